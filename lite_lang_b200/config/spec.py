@@ -46,10 +46,13 @@ class RunStep:
     layer's weights are then used again).  ``cache`` names the cache plane the
     mixer works on: ``None`` gives the entry a plane of its own; the index of
     an earlier entry makes it read that entry's plane without writing to it.
+    ``add_embedding``: the embedding's output is added to the residual before
+    the layer runs (a range of layers that runs again starts with it).
     """
 
     layer: int
     cache: Optional[int] = None
+    add_embedding: bool = False
 
 
 @dataclass(frozen=True)

@@ -75,14 +75,11 @@ extern "C" int ll_silu_mul(int dtype, void* out, const void* gate_up, int num_to
 }
 
 // ---------------------------------------------------------------------------------------------------------
-// The gated product with another activation: out[t, i] = act(gu[t, i]) * gu[t, I + i], act 0 SiLU, 1 ReLU.
+// The gated product with another activation (GateAct): out[t, i] of gate gu[t, i] and up gu[t, I + i].
 // ---------------------------------------------------------------------------------------------------------
-__device__ __forceinline__ float gate_activation(float g, int act) {
-  return act == 1 ? fmaxf(g, 0.f) : g / (1.0f + expf(-g));
-}
-
 template <typename T>
-__global__ void act_mul_kernel(T* __restrict__ out, const T* __restrict__ gu, long total, int inter, int act) {
+__global__ void act_mul_kernel(T* __restrict__ out, const T* __restrict__ gu, long total, int inter,
+                               const GateAct act) {
   LL_PDL_TRIGGER();
   LL_PDL_WAIT();
   const long idx0 = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -92,18 +89,18 @@ __global__ void act_mul_kernel(T* __restrict__ out, const T* __restrict__ gu, lo
     const int i = (int)(idx - t * inter);
     const float g = to_f32<T>(gu[t * 2 * inter + i]);
     const float u = to_f32<T>(gu[t * 2 * inter + inter + i]);
-    out[idx] = from_f32<T>(gate_activation(g, act) * u);
+    out[idx] = from_f32<T>(ll_gated(g, u, act));
   }
 }
 
 extern "C" int ll_act_mul(int dtype, void* out, const void* gate_up, int num_tokens, int inter, int act,
-                          cudaStream_t stream) {
+                          float limit, float alpha, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
-  if (act < 0 || act > 1) return (int)cudaErrorInvalidValue;
+  if (act < 0 || act > 2) return (int)cudaErrorInvalidValue;
   const long total = (long)num_tokens * inter;
   const int blocks = (int)min((total + 255) / 256, (long)silu_device_sms() * 16);
   LL_DISPATCH_DTYPE(dtype, ll_launch(act_mul_kernel<T>, dim3(blocks), dim3(256), 0, stream, (T*)out,
-                                     (const T*)gate_up, total, inter, act));
+                                     (const T*)gate_up, total, inter, (GateAct{act, limit, alpha})));
   return LL_LAUNCH_RESULT();
 }
 
@@ -211,5 +208,50 @@ extern "C" int ll_scale_f32(float* z, long total, float factor, cudaStream_t str
   if (total <= 0) return 0;
   const int blocks = (int)min((total + 255) / 256, (long)silu_device_sms() * 16);
   ll_launch(scale_f32_kernel, dim3(blocks), dim3(256), 0, stream, z, total, factor);
+  return LL_LAUNCH_RESULT();
+}
+
+// x[t, i] <- x[t, i] * sigmoid(gate[t, i]) in place; VEC neighbouring numbers of a row a thread (one 16-byte access).
+template <typename T, int VEC>
+__global__ void gate_rows_kernel(T* __restrict__ x, const T* __restrict__ gate, long gate_stride, long total_vec,
+                                 int width) {
+  LL_PDL_TRIGGER();
+  LL_PDL_WAIT();
+  const int per_row = width / VEC;
+  const long step = (long)gridDim.x * blockDim.x;
+  for (long idx = (long)blockIdx.x * blockDim.x + threadIdx.x; idx < total_vec; idx += step) {
+    const long t = idx / per_row;
+    const T* gp = gate + t * gate_stride + (idx - t * per_row) * VEC;
+    T* xp = x + idx * VEC;
+    T v[VEC], g[VEC];
+    if (VEC > 1) {
+      *reinterpret_cast<uint4*>(v) = *reinterpret_cast<const uint4*>(xp);
+      *reinterpret_cast<uint4*>(g) = *reinterpret_cast<const uint4*>(gp);
+    } else {
+      v[0] = xp[0];
+      g[0] = gp[0];
+    }
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) v[i] = from_f32<T>(to_f32<T>(v[i]) / (1.0f + expf(-to_f32<T>(g[i]))));
+    if (VEC > 1) *reinterpret_cast<uint4*>(xp) = *reinterpret_cast<const uint4*>(v);
+    else xp[0] = v[0];
+  }
+}
+
+extern "C" int ll_gate_rows(int dtype, void* x, const void* gate, long gate_stride, int num_tokens, int width,
+                            cudaStream_t stream) {
+  if (num_tokens <= 0) return 0;
+  if (width <= 0) return (int)cudaErrorInvalidValue;
+  const long most = (long)silu_device_sms() * 16;
+  LL_DISPATCH_DTYPE(dtype, {
+    constexpr int VEC = 16 / (int)sizeof(T);
+    const bool wide = width % VEC == 0 && gate_stride % VEC == 0 && (uintptr_t)x % 16 == 0 && (uintptr_t)gate % 16 == 0;
+    const long total = (long)num_tokens * width / (wide ? VEC : 1);
+    const dim3 grid((int)min((total + 255) / 256, most));
+    if (wide)
+      ll_launch(gate_rows_kernel<T, VEC>, grid, dim3(256), 0, stream, (T*)x, (const T*)gate, gate_stride, total, width);
+    else
+      ll_launch(gate_rows_kernel<T, 1>, grid, dim3(256), 0, stream, (T*)x, (const T*)gate, gate_stride, total, width);
+  });
   return LL_LAUNCH_RESULT();
 }

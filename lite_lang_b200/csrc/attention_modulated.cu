@@ -7,6 +7,7 @@
 //                                                                 ln(floor((p + 1) / every) + 1), optional
 //   raw_h[j] <- cap * tanh(raw_h[j] / cap)                        cap optional
 //   raw_h[j] <- raw_h[j] + rel[min(p - j, nd - 1), h]             rel optional: a bias by distance, [nd, nh]
+//   raw_h[j] <- raw_h[j] - slope[h] * (p - j)                     slope optional: a penalty by distance
 //   s_h[j]    = sum_g mix[h, g] raw_g[j]                          mix optional ([nh, nh], mixes all heads' scores)
 //   visible   : mask 0: j <= p;  1: p - j < size (a window) or j < keep (the request's first tokens stay
 //               visible);  2: j / size == p / size (chunks counted from position 0 of the request), always j <= p
@@ -37,7 +38,7 @@ attention_modulated_kernel(T* __restrict__ out, long out_stride, const T* __rest
                            const float* __restrict__ temp, const float* __restrict__ mix, int tk, int* status,
                            const float* __restrict__ sink_val, const float* __restrict__ rel, int nd, int keep,
                            float cap, float qt_coef, int qt_every, long gate_stride, int gate_channels,
-                           float out_scale) {
+                           float out_scale, const float* __restrict__ slope) {
   extern __shared__ float smem[];
   LL_PDL_WAIT();
   LL_PDL_TRIGGER();
@@ -125,6 +126,7 @@ attention_modulated_kernel(T* __restrict__ out, long out_stride, const T* __rest
         for (int d = 0; d < hd; ++d) s = fmaf(qh[d], kj[d], s);
         s *= (temp ? scale * temp[head0 + h] : scale) * qf;
         if (cap > 0.f) s = cap * tanhf(s / cap);
+        if (slope) s -= slope[head0 + h] * (float)(p - pos);
         if (rel && valid) s += rel[(size_t)min(p - pos, nd - 1) * nh + head0 + h];
       }
       raw[h * 32 + lane] = s;
@@ -216,7 +218,8 @@ extern "C" int ll_attention_modulated(int dtype, void* out, long out_stride, con
                                       int page_size, int num_pages, int mask, int mask_size, int sink, float scale,
                                       const float* temp, const float* mix, int* status, const float* sink_val,
                                       const float* rel, int nd, int keep, float cap, float qt_coef, int qt_every,
-                                      long gate_stride, int gate_channels, float out_scale, cudaStream_t stream) {
+                                      long gate_stride, int gate_channels, float out_scale, const float* slope,
+                                      cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (hd <= 0 || vd <= 0 || nkv <= 0 || nh % nkv != 0 || page_size <= 0 || mask < 0 || mask > 2 ||
       (rel != nullptr && nd <= 0) || keep < 0)
@@ -237,7 +240,7 @@ extern "C" int ll_attention_modulated(int dtype, void* out, long out_stride, con
               (const T*)q, q_stride, (const T*)gate, (const T*)k_cache, (const T*)v_cache, block_table, bt_stride,  \
               token_req, req_slot, positions, nh, nkv, hd, vd, page_size, num_pages, mask, mask_size, sink, scale,  \
               temp, mix, tk, status, sink_val, rel, nd, keep, cap, qt_coef, qt_every, gate_stride, gate_channels,   \
-              out_scale);                                                                                           \
+              out_scale, slope);                                                                                    \
   } while (0)
   LL_DISPATCH_DTYPE(dtype, {
     if (per_thread <= 4) AM_LAUNCH(4);

@@ -28,7 +28,8 @@
 // (1 + coef ln(floor((p + 1) / every) + 1)); a cap, s <- cap tanh(s / cap); a bias by distance from a table
 // [distances, heads], added after the cap; with a window, the request's first `keep` positions stay visible (the
 // stages that hold them are walked before the window's: by part 0 where the keys are split); a sink of a learned
-// score a head in the place of 0; a sigmoid gate a channel in the place of one a head; a constant on the output.
+// score a head in the place of 0; a sigmoid gate a channel in the place of one a head; a constant on the output; a
+// penalty that grows with the distance by a slope a head, taken off after the cap.
 #include "common.cuh"
 
 #define AS_WARPS 8
@@ -68,6 +69,7 @@ struct AttnShapedParams {
   int qt_every;           // > 0: the query's factor by position
   int gate_channels;      // the gate is a number a channel: token t, head h, channel d at gate[t * gate_stride + h * VD + d]
   float out_scale;
+  const float* slope;     // optional [nh]: a key n positions back has slope * n taken off its score (natural units)
 };
 #define AS_LOG2E 1.4426950408889634f
 // tanh from exp2 and a division: absolute error of a few 1e-7
@@ -181,9 +183,10 @@ __global__ void __launch_bounds__(AS_THREADS) attn_shaped_kernel(const AttnShape
     }
   }
   int posr[2], lor[2];
-  float sc[2];
+  float sc[2], slope_log2[2];
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
+    slope_log2[i] = p.slope ? p.slope[headr[i]] * AS_LOG2E : 0.f;
     posr[i] = ctx + tokr[i];
     lor[i] = as_first_visible(p.mask, p.mask_size, posr[i]);
     sc[i] = p.scale_log2 * ((!MIX && p.temp) ? p.temp[headr[i]] : 1.0f);
@@ -343,6 +346,7 @@ __global__ void __launch_bounds__(AS_THREADS) attn_shaped_kernel(const AttnShape
             float v = (s_acc[u][x] + s_odd[u][x]) * sc[i];
             if (p.cap_log2 > 0.f) v = p.cap_log2 * as_tanh(v * p.inv_cap_log2);
             if (p.rel) v = fmaf(bias_v[u][x], AS_LOG2E, v);
+            if (p.slope) v = fmaf(slope_log2[i], (float)(key0 + 8 * u + 2 * c + (x & 1) - posr[i]), v);
             if (boundary) {
               const int j = key0 + 8 * u + 2 * c + (x & 1);
               if (j > posr[i] || (j < lor[i] && j >= keep)) v = -INFINITY;
@@ -549,7 +553,7 @@ extern "C" long ll_attn_shaped_smem(int nkv, int hd, int vd, int mixed) {
 // out [tokens, nh * vd].  k_cache [pages, nkv, page_size, hd], v_cache [pages, nkv, page_size, vd].
 // cu_q, ctx_len, req_slot: the entries; row_blocks = sum over them of ceil(q_len * group / 128).
 // sink_val (optional float32 [nh]), rel (optional float32 [nd, nh]), keep, cap (0: none), qt_coef / qt_every
-// (0: none), gate_channels, out_scale: see the head of this file.
+// (0: none), gate_channels, out_scale, slope (optional float32 [nh]): see the head of this file.
 // mask 0 causal, 1 window, 2 chunks of mask_size.  nsplit > 1 (every entry brings one token): the keys of a
 // row are cut into parts of `span` stages of 64 keys; part float32 [tokens, nh, nsplit, vd + 2].
 extern "C" int ll_attn_shaped(void* out, long out_stride, const void* q, long q_stride, int mixed, const void* gate,
@@ -559,14 +563,14 @@ extern "C" int ll_attn_shaped(void* out, long out_stride, const void* q, long q_
                               int page_size, int num_pages, int mask, int mask_size, int sink, float scale, int nsplit,
                               int span, float* part, int* status, const float* sink_val, const float* rel, int nd,
                               int keep, float cap, float qt_coef, int qt_every, int gate_channels, float out_scale,
-                              cudaStream_t stream) {
+                              const float* slope, cudaStream_t stream) {
   if (row_blocks <= 0 || n_entries <= 0) return 0;
   const long smem = ll_attn_shaped_smem(nkv, hd, vd, mixed);
   if (smem == 0 || page_size % 16 != 0 || nh % nkv != 0 || nkv > 65535 || mask < 0 || mask > 2 ||
       (mask != 0 && mask_size <= 0) || nsplit < 1 || nsplit > 65535 || (nsplit > 1 && (part == nullptr || span < 1)))
     return (int)cudaErrorInvalidValue;
   if ((q_stride % 8) != 0 || (out_stride % 8) != 0 || (rel != nullptr && nd <= 0) || keep < 0 ||
-      (mixed && (rel != nullptr || cap > 0.f || sink_val != nullptr)))
+      (mixed && (rel != nullptr || cap > 0.f || sink_val != nullptr || slope != nullptr)))
     return (int)cudaErrorInvalidValue;
   AttnShapedParams p;
   p.q = (const bf16*)q;
@@ -607,6 +611,7 @@ extern "C" int ll_attn_shaped(void* out, long out_stride, const void* q, long q_
   p.qt_every = qt_every;
   p.gate_channels = gate_channels;
   p.out_scale = out_scale;
+  p.slope = slope;
   dim3 grid(row_blocks, nkv, nsplit);
 #define AS_LAUNCH(HD_, VD_, MIX_)                                                                                  \
   do {                                                                                                             \

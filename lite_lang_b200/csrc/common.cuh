@@ -74,6 +74,31 @@ __device__ __forceinline__ void set_status(int* status, int code) {
   if (status != nullptr) atomicCAS(status, 0, code);
 }
 
+// The activation of a gated product: 0 silu(g) u, 1 relu(g) u, 2 (clamped swish) a sigmoid(alpha a) (c + 1) with
+// a = min(g, limit), c = clamp(u, -limit, limit).
+struct GateAct {
+  int act;
+  float limit, alpha;
+};
+__device__ __forceinline__ float ll_clamped_swish(float g, float u, float limit, float alpha) {
+  const float a = fminf(g, limit);
+  const float c = fminf(fmaxf(u, -limit), limit);
+  return a / (1.0f + expf(-alpha * a)) * (c + 1.0f);
+}
+__device__ __forceinline__ float ll_gated(float g, float u, const GateAct& k) {
+  if (k.act == 2) return ll_clamped_swish(g, u, k.limit, k.alpha);
+  return (k.act == 1 ? fmaxf(g, 0.f) : g / (1.0f + expf(-g))) * u;
+}
+// x * rcp(y) and the fast exponential instead of the IEEE division and expf (see where it is used)
+__device__ __forceinline__ float ll_gated_fast(float g, float u, const GateAct& k) {
+  if (k.act == 2) {
+    const float a = fminf(g, k.limit);
+    const float c = fminf(fmaxf(u, -k.limit), k.limit);
+    return __fdividef(a, 1.0f + __expf(-k.alpha * a)) * (c + 1.0f);
+  }
+  return k.act == 1 ? fmaxf(g, 0.f) * u : __fdividef(g, 1.0f + __expf(-g)) * u;
+}
+
 #define LL_DISPATCH_DTYPE(dtype, ...)              \
   do {                                             \
     if ((dtype) == LL_DTYPE_F32) {                 \

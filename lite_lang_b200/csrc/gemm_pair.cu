@@ -173,7 +173,8 @@ struct GpParams {
   int m_tiles;      // tiles of 256 tokens
   int tiles;        // m_tiles x column tiles (plain: 256 features a tile, gated: 128)
   int vec_ok;       // the output takes 16-byte pieces (aligned base and stride, N a multiple of 8)
-  int act;          // gated: 0 silu(gate) * up, 1 relu(gate) * up; plain: 0 none, 1 gelu (tanh form), 2 ReLU, 3 SiLU, 4 ReLU squared
+  GateAct gate;     // gated: the activation
+  int act;          // plain: 0 none, 1 gelu (tanh form), 2 ReLU, 3 SiLU, 4 ReLU squared
   int* status;
   // q|k|v mode only: what follows the projection (N = (nh + 2 nkv) hd; out is q [M, nh hd])
   const float* bias;      // float32 [N] or null
@@ -507,7 +508,7 @@ gemm_pair_kernel(const GpParams p, const __grid_constant__ CUtensorMap wmap, con
               const float uv = __bfloat162float(__float2bfloat16_rn(__uint_as_float(u[i])));
               // (x * rcp(y) instead of the IEEE division: that one's chain of dependent instructions with a
               //  branch an element, on the one warp a scheduler has here, made the epilogue twice as long as the MMAs)
-              v[i] = p.act ? fmaxf(gt, 0.f) * uv : __fdividef(gt, 1.0f + __expf(-gt)) * uv;
+              v[i] = ll_gated_fast(gt, uv, p.gate);
             }
           } else {
             unsigned a[32];
@@ -648,7 +649,7 @@ static int gp_launch(GpParams& p, const void* w, const void* x, long x_stride, i
 // x: bfloat16 [M, K] (row stride x_stride, a multiple of 8); w: bfloat16 [N, K] contiguous (gated: [2 N, K],
 // gate rows first); out: bfloat16 [M, N] (gated: silu(gate) * up).  Any M; meant for hundreds of tokens and more.
 extern "C" int ll_gemm_pair(void* out, long out_stride, const void* x, long x_stride, const void* w, int M, int N,
-                            int K, int gated, int sm_count, int* status, cudaStream_t stream) {
+                            int K, int gated, int sm_count, float limit, float alpha, int* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (K <= 0 || (K % 8) != 0 || (x_stride % 8) != 0 || sm_count < 2) return (int)cudaErrorInvalidValue;
   GpParams p;
@@ -658,7 +659,9 @@ extern "C" int ll_gemm_pair(void* out, long out_stride, const void* x, long x_st
   p.N = N;
   p.K = K;
   p.status = status;
-  p.act = gated == 2 ? 1 : 0;      // (gated: 1 SiLU, 2 ReLU)
+  if (gated < 0 || gated > 3) return (int)cudaErrorInvalidValue;
+  p.gate = {gated > 0 ? gated - 1 : 0, limit, alpha};      // (gated: 1 SiLU, 2 ReLU, 3 clamped swish)
+  p.act = 0;
   p.vec_ok = ((uintptr_t)out % 16 == 0 && out_stride % 8 == 0 && N % 8 == 0) ? 1 : 0;
   p.bias = nullptr;
   p.positions = nullptr;
@@ -685,6 +688,7 @@ extern "C" int ll_gemm_pair_act(void* out, long out_stride, const void* x, long 
   p.N = N;
   p.K = K;
   p.status = status;
+  p.gate = {0, 0.f, 0.f};
   p.act = act;
   p.vec_ok = ((uintptr_t)out % 16 == 0 && out_stride % 8 == 0 && N % 8 == 0) ? 1 : 0;
   p.bias = nullptr;
@@ -719,6 +723,7 @@ extern "C" int ll_gemm_pair_qkv_rope(void* q_out, long q_stride, const void* x, 
   p.N = (nh + 2 * nkv) * hd;
   p.K = K;
   p.status = status;
+  p.gate = {0, 0.f, 0.f};
   p.act = 0;
   p.vec_ok = 1;
   p.bias = bias;

@@ -50,8 +50,8 @@ template <> __device__ __forceinline__ bf16 gs_out<bf16>(float v) { return __flo
 template <int MT, bool GATED, typename OutT>
 __global__ void __launch_bounds__(GS_THREADS)
 gemm_smallm_kernel(OutT* __restrict__ out, long out_stride, const bf16* __restrict__ x, long x_stride,
-                   const bf16* __restrict__ w, int M, int N, int K, int act) {
-  // N is the number of output features (act: the gate's activation, 0 SiLU, 1 ReLU) (for GATED: the intermediate size I; W has 2 I rows)
+                   const bf16* __restrict__ w, int M, int N, int K, const GateAct act) {
+  // N is the number of output features (for GATED: the intermediate size I; W has 2 I rows)
   extern __shared__ float red[];  // [GS_WARPS][GATED ? 2 : 1][16][8 * MT]
   constexpr int TOK = 8 * MT;
   constexpr int NACC = GATED ? 2 : 1;
@@ -149,7 +149,7 @@ gemm_smallm_kernel(OutT* __restrict__ out, long out_stride, const bf16* __restri
       // rounded to the storage type first, as the unfused path does between the product and the activation
       const float gt = __bfloat162float(__float2bfloat16_rn(v[0]));
       const float up = __bfloat162float(__float2bfloat16_rn(v[NACC - 1]));
-      y = (act ? fmaxf(gt, 0.f) : gt / (1.0f + expf(-gt))) * up;
+      y = ll_gated(gt, up, act);
     }
     out[(size_t)tok * out_stride + f0 + f] = gs_out<OutT>(y);
   }
@@ -157,7 +157,7 @@ gemm_smallm_kernel(OutT* __restrict__ out, long out_stride, const bf16* __restri
 
 template <int MT, bool GATED, typename OutT>
 static int gs_launch(void* out, long out_stride, const void* x, long x_stride, const void* w, int M, int N, int K,
-                     int act, cudaStream_t stream) {
+                     GateAct act, cudaStream_t stream) {
   const size_t smem = sizeof(float) * GS_WARPS * (GATED ? 2 : 1) * 16 * 8 * MT;
   if (smem > 48 * 1024)
     cudaFuncSetAttribute(gemm_smallm_kernel<MT, GATED, OutT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -168,7 +168,7 @@ static int gs_launch(void* out, long out_stride, const void* x, long x_stride, c
 
 template <bool GATED, typename OutT>
 static int gs_dispatch_m(void* out, long out_stride, const void* x, long x_stride, const void* w, int M, int N, int K,
-                         int act, cudaStream_t stream) {
+                         GateAct act, cudaStream_t stream) {
   if (M <= 8) return gs_launch<1, GATED, OutT>(out, out_stride, x, x_stride, w, M, N, K, act, stream);
   if (M <= 16) return gs_launch<2, GATED, OutT>(out, out_stride, x, x_stride, w, M, N, K, act, stream);
   if (M <= 32) return gs_launch<4, GATED, OutT>(out, out_stride, x, x_stride, w, M, N, K, act, stream);
@@ -179,10 +179,11 @@ static int gs_dispatch_m(void* out, long out_stride, const void* x, long x_strid
 // x: bfloat16 [M, K] (row stride x_stride), w: bfloat16 [N, K] contiguous (gated: [2 N, K],
 // gate rows first), out: [M, N] bfloat16 (out_f32 = 0) or float32 (out_f32 = 1).
 extern "C" int ll_gemm_smallm(void* out, long out_stride, int out_f32, const void* x, long x_stride, const void* w,
-                              int M, int N, int K, int gated, cudaStream_t stream) {
+                              int M, int N, int K, int gated, float limit, float alpha, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 64 || K <= 0 || (K % 32) != 0 || (x_stride % 8) != 0) return (int)cudaErrorInvalidValue;
-  const int act = gated == 2 ? 1 : 0;      // (gated: 1 SiLU, 2 ReLU)
+  if (gated < 0 || gated > 3) return (int)cudaErrorInvalidValue;
+  const GateAct act = {gated > 0 ? gated - 1 : 0, limit, alpha};      // (gated: 1 SiLU, 2 ReLU, 3 clamped swish)
   if (gated) {
     if (out_f32) return (int)cudaErrorInvalidValue;
     return gs_dispatch_m<true, bf16>(out, out_stride, x, x_stride, w, M, N, K, act, stream);

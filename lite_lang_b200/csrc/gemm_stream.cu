@@ -154,7 +154,7 @@ struct GtParams {
   int units;    // feature units times ksplit
   int ksplit;   // parts the k range is cut into; > 1: out is float32 [ksplit, M, N] partial sums
   int cpp;      // k chunks (stages) per part
-  int act;      // GATED: 0 silu(gate) * up, 1 relu(gate) * up
+  GateAct gate; // GATED: the activation
   int row_act;  // WIDE to bfloat16 with k whole: 0 none; 1 gelu (tanh form), 2 ReLU, 3 SiLU, 4 ReLU squared on the result, which is
                 // rounded to bfloat16 first, as a product followed by an activation kernel would have it
   // QKV_ROPE only: what follows the projection
@@ -491,7 +491,7 @@ gemm_stream_kernel(const GtParams p, const __grid_constant__ CUtensorMap wmap, c
               const float rs = SPLIT ? row_scale[t] : 1.0f;
               const float gt = __bfloat162float(__float2bfloat16_rn(acc[j][h] * rs));
               const float up = __bfloat162float(__float2bfloat16_rn(acc[j][2 + h] * rs));
-              out[(size_t)t * p.out_stride + f] = gt_out<OutT>((p.act ? fmaxf(gt, 0.f) : gt / (1.0f + expf(-gt))) * up);
+              out[(size_t)t * p.out_stride + f] = gt_out<OutT>(ll_gated(gt, up, p.gate));
             }
           }
         }
@@ -674,10 +674,10 @@ static int gt_dispatch_m(const GtParams& p, const void* w, int sm_count, cudaStr
 // sums that the caller adds (the fused residual-and-norm kernel does).
 // sm_count: SMs of the device (the grid is at most two CTAs an SM).
 extern "C" int ll_gemm_stream(void* out, long out_stride, int out_f32, const void* x, long x_stride, const void* w,
-                              int M, int N, int K, int mode, int ksplit, int sm_count, int* status,
-                              cudaStream_t stream) {
+                              int M, int N, int K, int mode, int ksplit, int sm_count, float limit, float alpha,
+                              int* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
-  const int act = (mode >> 8) & 0xff;        // (bits 8..15: the gated mode's activation, 0 SiLU, 1 ReLU)
+  const int act = (mode >> 8) & 0xff;        // (bits 8..15: the gated mode's activation, see GateAct; its limit and alpha)
   const int row_act = (mode >> 16) & 0xff;   // (bits 16..23: an activation on the wide mode's result, see GtParams)
   mode &= 0xff;
   if (row_act != 0 && (mode != GT_MODE_WIDE || out_f32 || ksplit != 1 || row_act > 4)) return (int)cudaErrorInvalidValue;
@@ -693,7 +693,8 @@ extern "C" int ll_gemm_stream(void* out, long out_stride, int out_f32, const voi
   p.M = M;
   p.N = N;
   p.K = K;
-  p.act = act == 1 ? 1 : 0;
+  if (act > 2) return (int)cudaErrorInvalidValue;
+  p.gate = {act, limit, alpha};
   p.row_act = row_act;
   p.status = status;
   if (mode == GT_MODE_WIDE) {

@@ -102,7 +102,7 @@ struct TcParams {
   int ksplit;    // > 1: out is float32 [ksplit, M, N] partial sums
   int cpp;       // 64-wide k boxes per part
   int vec_ok;    // the output takes 16-byte pieces (aligned base and stride, N a multiple of the piece)
-  int act;       // gated: 0 silu(gate) * up, 1 relu(gate) * up
+  GateAct gate;  // gated: the activation
   // SCALED (gated, at most 64 tokens): the tokens' rows are only multiplied by the weight of the norm before this
   // product yet; the rows' sums of squares come in parts [sumsq_units][64] (see gemm_stream.cu: the product before
   // the norm leaves them), and each row of the result is scaled by 1 / sqrt(sum / K + eps) before the activation
@@ -327,7 +327,7 @@ gemm_tc_kernel(const TcParams p, const __grid_constant__ CUtensorMap wmap, const
           const float gt = __bfloat162float(__float2bfloat16_rn(a * rs));
           const float uv = __bfloat162float(__float2bfloat16_rn(stg[(64 + fl) * (NT + 1) + t] * rs));
           // (x * rcp(y), not the IEEE division: that is a chain of dependent instructions with a branch an element)
-          return p.act ? fmaxf(gt, 0.f) * uv : __fdividef(gt, 1.0f + __expf(-gt)) * uv;
+          return ll_gated_fast(gt, uv, p.gate);
         }
         return a;
       };
@@ -429,7 +429,7 @@ static int tc_launch(const TcParams& p, const void* w, const void* x, long x_str
 // sumsq (gated, M <= 64; or null): see TcParams.
 extern "C" int ll_gemm_tc(void* out, long out_stride, int out_f32, const void* x, long x_stride, const void* w, int M,
                           int N, int K, int gated, int ksplit, int sm_count, const float* sumsq, int sumsq_units,
-                          float norm_eps, int* status, cudaStream_t stream) {
+                          float norm_eps, float limit, float alpha, int* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (sumsq != nullptr && (!gated || M > 64 || sumsq_units <= 0)) return (int)cudaErrorInvalidValue;
   if (M > 128 || K <= 0 || (K % 64) != 0 || (x_stride % 8) != 0 || sm_count <= 0 || ksplit < 1)
@@ -442,7 +442,8 @@ extern "C" int ll_gemm_tc(void* out, long out_stride, int out_f32, const void* x
   p.N = N;
   p.K = K;
   p.status = status;
-  p.act = gated == 2 ? 1 : 0;      // (gated: 1 SiLU, 2 ReLU)
+  if (gated < 0 || gated > 3) return (int)cudaErrorInvalidValue;
+  p.gate = {gated > 0 ? gated - 1 : 0, limit, alpha};      // (gated: 1 SiLU, 2 ReLU, 3 clamped swish)
   p.sumsq_in = sumsq;
   p.sumsq_units = sumsq_units;
   p.norm_eps = norm_eps;

@@ -8,8 +8,8 @@
 // cached rows, its values the first R numbers of the same rows, and what it returns is sum_j p_j c_j per head
 // (expanded by a batched product after it).  Nothing per head is ever cached or re-expanded.
 //
-// Rotation (interleaved pairs): numbers 2i and 2i+1 of a rotated part, for 2i < rot_dims, turn by the angle
-// position * freq[i]; (u, v) -> (u cos - v sin, v cos + u sin); the rest passes unchanged.  Angles, the
+// Rotation: numbers 2i and 2i+1 (interleaved pairs) or i and i + rot_dims / 2 (half-split pairs) of a rotated part, for
+// i < rot_dims / 2, turn by the angle position * freq[i]; (u, v) -> (u cos - v sin, v cos + u sin); the rest passes.  Angles, the
 // latent's norm, scores and softmax are float32.
 //
 //   latent_prepare    per token: RMS norm of the latent, rotation of k_r and of every head's q_r, cache write
@@ -23,6 +23,21 @@
 // every sum depends on the position only, not on how the tokens were cut into steps or batched.
 #include "common.cuh"
 
+// number j of a rotated part whose numbers are src[0 .. r)
+template <typename T>
+__device__ __forceinline__ float la_rotated(const T* src, int j, float p, const float* freq, int half, int half_split,
+                                            float amplitude) {
+  if (j >= 2 * half) return to_f32<T>(src[j]);
+  const int i = half_split ? (j < half ? j : j - half) : j >> 1;            // the pair, its first and its second number
+  const int iu = half_split ? i : 2 * i, iv = half_split ? i + half : 2 * i + 1;
+  float sn, cs;
+  sincosf(p * freq[i], &sn, &cs);
+  sn *= amplitude;
+  cs *= amplitude;
+  const float u = to_f32<T>(src[iu]), v = to_f32<T>(src[iv]);
+  return j == iv ? v * cs + u * sn : u * cs - v * sn;
+}
+
 // qsrc row t (row stride q_stride; the projection itself, or the output of a second product when the queries go
 // through a latent of their own): q heads at q_off, head h's rotated part at q_off + h * (d + r) + d; proj row t:
 // the latent at kv_off (R wide), then the rotated key part (r wide).  Both cos and sin are multiplied by
@@ -33,7 +48,7 @@ latent_prepare_kernel(const T* __restrict__ proj, long proj_stride, int q_off, i
                       float eps, const float* __restrict__ freq, int rot_dims, const int* __restrict__ positions,
                       const int* __restrict__ slot_map, T* __restrict__ cache, long num_slots,
                       T* __restrict__ q_full, int H, int d, int r, int R, int* status, float amplitude,
-                      const T* __restrict__ qsrc, long q_stride) {
+                      const T* __restrict__ qsrc, long q_stride, int half_split) {
   __shared__ float scratch[32];
   LL_PDL_TRIGGER();
   LL_PDL_WAIT();
@@ -45,17 +60,7 @@ latent_prepare_kernel(const T* __restrict__ proj, long proj_stride, int q_off, i
   for (int i = tid; i < H * r; i += blockDim.x) {
     const int h = i / r, j = i % r;
     const T* src = qsrc + (size_t)t * q_stride + q_off + (size_t)h * (d + r) + d;
-    float out;
-    if (j < 2 * half) {
-      float sn, cs;
-      sincosf(p * freq[j >> 1], &sn, &cs);
-      sn *= amplitude;
-      cs *= amplitude;
-      const float u = to_f32<T>(src[j & ~1]), v = to_f32<T>(src[j | 1]);
-      out = (j & 1) ? v * cs + u * sn : u * cs - v * sn;
-    } else {
-      out = to_f32<T>(src[j]);
-    }
+    const float out = la_rotated<T>(src, j, p, freq, half, half_split, amplitude);
     q_full[((size_t)t * H + h) * (R + r) + R + j] = from_f32<T>(out);
   }
   const long slot = slot_map ? slot_map[t] : -1;
@@ -74,20 +79,8 @@ latent_prepare_kernel(const T* __restrict__ proj, long proj_stride, int q_off, i
   const float inv = 1.0f / sqrtf(ss / (float)R + eps);
   T* dst = cache + (size_t)slot * (R + r);
   for (int i = tid; i < R; i += blockDim.x) dst[i] = from_f32<T>(to_f32<T>(lat[i]) * inv * norm_w[i]);
-  for (int j = tid; j < r; j += blockDim.x) {
-    float out;
-    if (j < 2 * half) {
-      float sn, cs;
-      sincosf(p * freq[j >> 1], &sn, &cs);
-      sn *= amplitude;
-      cs *= amplitude;
-      const float u = to_f32<T>(lat[R + (j & ~1)]), v = to_f32<T>(lat[R + (j | 1)]);
-      out = (j & 1) ? v * cs + u * sn : u * cs - v * sn;
-    } else {
-      out = to_f32<T>(lat[R + j]);
-    }
-    dst[R + j] = from_f32<T>(out);
-  }
+  for (int j = tid; j < r; j += blockDim.x)
+    dst[R + j] = from_f32<T>(la_rotated<T>(lat + R, j, p, freq, half, half_split, amplitude));
 }
 
 #define LA_TK 32
@@ -499,13 +492,13 @@ extern "C" int ll_latent_prepare(int dtype, const void* proj, long proj_stride, 
                                  const float* norm_w, float eps, const float* freq, int rot_dims, const int* positions,
                                  const int* slot_map, void* cache, long num_slots, void* q_full, int num_tokens, int H,
                                  int d, int r, int R, int* status, float amplitude, const void* qsrc, long q_stride,
-                                 cudaStream_t stream) {
+                                 int half_split, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (H <= 0 || d < 0 || r < 0 || R <= 0 || rot_dims < 0 || rot_dims > r) return (int)cudaErrorInvalidValue;
   LL_DISPATCH_DTYPE(dtype, ll_launch(latent_prepare_kernel<T>, dim3(num_tokens), dim3(128), 0, stream, (const T*)proj,
                                      proj_stride, q_off, kv_off, norm_w, eps, freq, rot_dims, positions, slot_map,
                                      (T*)cache, num_slots, (T*)q_full, H, d, r, R, status, amplitude,
-                                     (const T*)qsrc, q_stride));
+                                     (const T*)qsrc, q_stride, half_split));
   return LL_LAUNCH_RESULT();
 }
 

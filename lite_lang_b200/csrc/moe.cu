@@ -1,8 +1,10 @@
 // Routed feed-forward (mixture of experts): the router and the activation between the two products.
 //
 // Router, per token, all in float32: logits z = Wr x over the experts, scores by softmax (or sigmoid) over
-// all experts, the `top` experts with the largest scores (ties: the lower index), their weights the scores
-// themselves or the scores divided by their sum.  The result is a dense row of weights per token, zero for
+// all experts, the `top` experts with the largest choice scores (ties: the lower index; the choice scores are the
+// scores, or the scores plus a number an expert that the weights do not see), their weights the scores
+// themselves or the scores divided by their sum, times a constant.  The choice may be kept to the best groups of
+// neighbouring experts.  Outputs of the router beyond the experts stand for the token's row itself (identities).  The result is a dense row of weights per token, zero for
 // experts that were not chosen, plus the chosen indices and weights.
 //
 // The experts' first products run as one product over all experts' rows (an always-on expert's rows first);
@@ -17,7 +19,11 @@
 // [tokens, top].  score_fn: 0 softmax over all experts, 1 sigmoid, 2 the `top` largest logits are chosen and
 // their weights are a softmax taken over just those logits.  `bias` (float32 [E], optional) is added to the
 // logits.  With `shared_w` (float32 [tokens]) the router matrix has one more row, the gate of an expert that
-// every token uses: shared_w[t] = sigmoid(Wr[E] . x).  One block per token: its eight warps share out the experts
+// every token uses: shared_w[t] = sigmoid(Wr[E] . x).  E counts all outputs of the router; `gates` has `real` columns,
+// and outputs real .. E - 1 are identities, whose weights add up to identity_w[t].  choice_bias (float32 [E], optional)
+// is added to the scores for the choice.  With `keep` < `count`, only outputs of the `keep` groups (E / count neighbours
+// each) with the largest best choice score can be chosen.  A place that finds nothing left gets top_idx -1 and weight 0.
+// One block per token: its eight warps share out the experts
 // (the token's row waits in shared memory as float32), then the first warp scores and picks.
 #define MOE_ROUTER_THREADS 256
 template <typename T>
@@ -25,8 +31,11 @@ __global__ void __launch_bounds__(MOE_ROUTER_THREADS)
 moe_router_kernel(const T* __restrict__ x, long x_stride, const float* __restrict__ Wr, const float* __restrict__ bias,
                   float* __restrict__ gates, int* __restrict__ top_idx, float* __restrict__ top_w,
                   float* __restrict__ shared_w, int num_tokens, int hidden, int E, int top, int score_fn,
-                  int renormalize) {
+                  int renormalize, const float* __restrict__ choice_bias, int count, int keep, float weight_scale,
+                  float* __restrict__ identity_w, int real) {
   __shared__ float z[MOE_MAX_E + 2];
+  __shared__ float cs[MOE_MAX_E];                        // choice scores
+  __shared__ float gb[MOE_MAX_E];                        // the groups' best
   extern __shared__ __align__(16) float xrow[];          // the token's row as float32 [hidden]
   LL_PDL_TRIGGER();
   LL_PDL_WAIT();
@@ -76,15 +85,33 @@ moe_router_kernel(const T* __restrict__ x, long x_stride, const float* __restric
     for (int e = lane; e < E; e += 32) z[e] = 1.0f / (1.0f + expf(-z[e]));
   }
   __syncwarp();
-  float* gr = gates + (size_t)t * E;
-  for (int e = lane; e < E; e += 32) gr[e] = 0.f;
+  float* gr = gates + (size_t)t * real;
+  for (int e = lane; e < real; e += 32) gr[e] = 0.f;
+  for (int e = lane; e < E; e += 32) cs[e] = z[e] + (choice_bias ? choice_bias[e] : 0.f);
   __syncwarp();
-  float total = 0.f;
+  if (keep < count) {
+    const int size = E / count;
+    for (int g = lane; g < count; g += 32) {
+      float best = -INFINITY;
+      for (int e = g * size; e < (g + 1) * size; ++e) best = fmaxf(best, cs[e]);
+      gb[g] = best;
+    }
+    __syncwarp();
+    // a group is out if at least `keep` groups are better (among equals the lower index is)
+    for (int g = lane; g < count; g += 32) {
+      int better = 0;
+      for (int o = 0; o < count; ++o) better += (gb[o] > gb[g] || (gb[o] == gb[g] && o < g)) ? 1 : 0;
+      if (better >= keep)
+        for (int e = g * size; e < (g + 1) * size; ++e) cs[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  float total = 0.f, ident = 0.f;
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
     int arg = E;
     for (int e = lane; e < E; e += 32) {
-      const float v = z[e];
+      const float v = cs[e];
       if (v > best) {   // (a lane walks upwards, so it keeps its lowest index among equals)
         best = v;
         arg = e;
@@ -99,16 +126,25 @@ moe_router_kernel(const T* __restrict__ x, long x_stride, const float* __restric
         arg = oa;
       }
     }
-    if (arg >= E) break;
+    if (arg >= E) {       // nothing left to choose
+      if (lane == 0) {
+        top_idx[(size_t)t * top + k] = -1;
+        top_w[(size_t)t * top + k] = 0.f;
+      }
+      continue;
+    }
+    const float w = z[arg] * weight_scale;
     if (lane == 0) {
       top_idx[(size_t)t * top + k] = arg;
-      top_w[(size_t)t * top + k] = best;
-      gr[arg] = best;
-      z[arg] = -INFINITY;
+      top_w[(size_t)t * top + k] = w;
+      if (arg < real) gr[arg] = w;
+      cs[arg] = -INFINITY;
     }
-    total += best;
+    if (arg >= real) ident += w;
+    total += z[arg];
     __syncwarp();
   }
+  if (identity_w && lane == 0) identity_w[t] = (renormalize && total > 0.f) ? ident / total : ident;
   if (score_fn == 2) {
     // softmax over the chosen logits (the first chosen is the largest), summed in the order they were chosen
     __syncwarp();
@@ -125,7 +161,7 @@ moe_router_kernel(const T* __restrict__ x, long x_stride, const float* __restric
   }
   if (renormalize && total > 0.f) {
     __syncwarp();
-    for (int e = lane; e < E; e += 32) gr[e] = gr[e] / total;
+    for (int e = lane; e < real; e += 32) gr[e] = gr[e] / total;
     for (int k = lane; k < top; k += 32) top_w[(size_t)t * top + k] /= total;
   }
 }
@@ -191,14 +227,18 @@ __global__ void moe_act_kernel(T* __restrict__ h, const float* __restrict__ gate
 
 extern "C" int ll_moe_router(int dtype, const void* x, long x_stride, const float* Wr, const float* bias, float* gates,
                              int* top_idx, float* top_w, float* shared_w, int num_tokens, int hidden, int E, int top,
-                             int score_fn, int renormalize, cudaStream_t stream) {
+                             int score_fn, int renormalize, const float* choice_bias, int count, int keep,
+                             float weight_scale, float* identity_w, int real, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
+  if (real <= 0 || real > E || (real < E && identity_w == nullptr) || count < 1 || E % count != 0 || keep < 1 || keep > count)
+    return (int)cudaErrorInvalidValue;
   if (E <= 0 || E > MOE_MAX_E || top <= 0 || top > E || hidden <= 0) return (int)cudaErrorInvalidValue;
   const size_t smem = sizeof(float) * (size_t)((hidden + 3) / 4 * 4);
   if (smem > 40 * 1024) return (int)cudaErrorInvalidValue;      // (rows of up to 10,240 numbers)
   LL_DISPATCH_DTYPE(dtype, ll_launch(moe_router_kernel<T>, dim3(num_tokens), dim3(MOE_ROUTER_THREADS), smem, stream,
                                      (const T*)x, x_stride, Wr, bias, gates, top_idx, top_w, shared_w, num_tokens,
-                                     hidden, E, top, score_fn, renormalize));
+                                     hidden, E, top, score_fn, renormalize, choice_bias, count, keep, weight_scale,
+                                     identity_w, real));
   return LL_LAUNCH_RESULT();
 }
 
@@ -241,6 +281,7 @@ moe_sort_kernel(const int* __restrict__ top_idx, const float* __restrict__ top_w
                 int* __restrict__ pair_row) {
   __shared__ int count[MOE_MAX_E];
   __shared__ int start[MOE_MAX_E];
+  __shared__ int used;
   LL_PDL_WAIT();      // (no early release: what runs next may be a library kernel that does not wait itself)
   for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 1;
   __syncthreads();
@@ -258,8 +299,14 @@ moe_sort_kernel(const int* __restrict__ top_idx, const float* __restrict__ top_w
       at += count[e];
       ends[e] = at;
     }
+    used = at;
   }
   __syncthreads();
+  // rows behind the last run (pairs that no expert has: identities): a token that exists, weight 0
+  for (int row = used + threadIdx.x; row < pairs + E; row += blockDim.x) {
+    row_token[row] = 0;
+    row_w[row] = 0.f;
+  }
   for (int p = threadIdx.x; p < pairs; p += blockDim.x) {
     const int e = top_idx[p];
     if (e >= 0 && e < E) {
@@ -368,51 +415,63 @@ extern "C" int ll_moe_combine(int dtype, void* out, const void* base, const void
 
 // ---------------------------------------------------------------------------------------------------------
 // Experts with a gate: an expert is down(a * sigmoid(alpha a) * (c + 1)) with a = min(gate x, limit) and
-// c = clamp(up x, -limit, limit).  The first product's rows are, expert by expert, the gate rows then the up
+// c = clamp(up x, -limit, limit), or (a limit of 0) down(silu(gate x) * (up x)).  The first product's rows are, expert by expert, the gate rows then the up
 // rows (an always-on expert's first).
 // ---------------------------------------------------------------------------------------------------------
-__device__ __forceinline__ float clamped_swish_gate(float g, float u, float limit, float alpha) {
-  const float a = fminf(g, limit);
-  const float c = fminf(fmaxf(u, -limit), limit);
-  return a / (1.0f + expf(-alpha * a)) * (c + 1.0f);
+__device__ __forceinline__ float moe_gate(float g, float u, float limit, float alpha) {
+  return limit > 0.f ? ll_clamped_swish(g, u, limit, alpha) : g / (1.0f + expf(-g)) * u;
 }
 
 // in: T [tokens, 2 * (shared_ff + E * ff)]; out: T [tokens, shared_ff + E * ff] = activation times the
 // expert's weight for the token: gates[t, e] for expert e (zero: not chosen, zeros are written and nothing is
 // read), shared_w[t] (null: 1) for the always-on expert, which has a limit of its own.
-template <typename T>
+// A thread takes VEC neighbouring units (one 16-byte access where the widths allow it: they lie inside one expert then).
+template <typename T, int VEC>
 __global__ void moe_gated_act_kernel(T* __restrict__ out, const T* __restrict__ in, const float* __restrict__ gates,
                                      const float* __restrict__ shared_w, int num_tokens, int shared_ff, int ff, int E,
                                      float limit, float shared_limit, float alpha) {
   LL_PDL_TRIGGER();
   LL_PDL_WAIT();
   const int width = shared_ff + E * ff;
-  const long total = (long)num_tokens * width;
+  const int per_row = width / VEC;
+  const long total = (long)num_tokens * per_row;
   const long step = (long)gridDim.x * blockDim.x;
   for (long idx = (long)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += step) {
-    const int t = (int)(idx / width);
-    const int c = (int)(idx - (long)t * width);
+    const int t = (int)(idx / per_row);
+    const int c = (int)(idx - (long)t * per_row) * VEC;
     const T* row = in + (size_t)t * 2 * width;
-    float w, g, u, lim;
+    T* dst = out + (size_t)t * width + c;
+    float w, lim;
+    const T *gp, *up;
+    T g[VEC], u[VEC], y[VEC];
     if (c < shared_ff) {
       w = shared_w ? shared_w[t] : 1.f;
-      g = to_f32<T>(row[c]);
-      u = to_f32<T>(row[shared_ff + c]);
+      gp = row + c;
+      up = gp + shared_ff;
       lim = shared_limit;
     } else {
       const int e = (c - shared_ff) / ff;
-      const int j = (c - shared_ff) - e * ff;
       w = gates[(size_t)t * E + e];
+      gp = row + 2 * shared_ff + (size_t)e * 2 * ff + (c - shared_ff - e * ff);
+      up = gp + ff;
+      lim = limit;
       if (w == 0.f) {      // an expert that was not chosen contributes an exact zero whatever its first product gave
-        out[idx] = from_f32<T>(0.f);
+        if (VEC > 1) *reinterpret_cast<uint4*>(dst) = make_uint4(0, 0, 0, 0);
+        else dst[0] = from_f32<T>(0.f);
         continue;
       }
-      const T* p = row + 2 * shared_ff + (size_t)e * 2 * ff;
-      g = to_f32<T>(p[j]);
-      u = to_f32<T>(p[ff + j]);
-      lim = limit;
     }
-    out[idx] = from_f32<T>(clamped_swish_gate(g, u, lim, alpha) * w);
+    if (VEC > 1) {
+      *reinterpret_cast<uint4*>(g) = *reinterpret_cast<const uint4*>(gp);
+      *reinterpret_cast<uint4*>(u) = *reinterpret_cast<const uint4*>(up);
+    } else {
+      g[0] = gp[0];
+      u[0] = up[0];
+    }
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) y[k] = from_f32<T>(moe_gate(to_f32<T>(g[k]), to_f32<T>(u[k]), lim, alpha) * w);
+    if (VEC > 1) *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(y);
+    else dst[0] = y[0];
   }
 }
 
@@ -439,7 +498,7 @@ __global__ void moe_row_gated_act_kernel(T* __restrict__ out, const T* __restric
     }
 #pragma unroll
     for (int k = 0; k < VEC; ++k)
-      y[k] = from_f32<T>(clamped_swish_gate(to_f32<T>(g[k]), to_f32<T>(u[k]), limit, alpha) * w);
+      y[k] = from_f32<T>(moe_gate(to_f32<T>(g[k]), to_f32<T>(u[k]), limit, alpha) * w);
     if (VEC > 1) *reinterpret_cast<uint4*>(out + (size_t)r * ff + j) = *reinterpret_cast<const uint4*>(y);
     else out[(size_t)r * ff + j] = y[0];
   }
@@ -449,12 +508,21 @@ extern "C" int ll_moe_gated_act(int dtype, void* out, const void* in, const floa
                                 int num_tokens, int shared_ff, int ff, int E, float limit, float shared_limit,
                                 float alpha, int sms, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
-  const long total = (long)num_tokens * (shared_ff + (long)E * ff);
-  if (total <= 0) return (int)cudaErrorInvalidValue;
-  const long most = (long)(sms > 0 ? sms : 148) * 16, want = (total + 255) / 256;
-  LL_DISPATCH_DTYPE(dtype, ll_launch(moe_gated_act_kernel<T>, dim3((int)(want < most ? want : most)), dim3(256), 0,
-                                     stream, (T*)out, (const T*)in, gates, shared_w, num_tokens, shared_ff, ff, E,
-                                     limit, shared_limit, alpha));
+  const long width = shared_ff + (long)E * ff;
+  if (width <= 0 || (E > 0 && ff <= 0)) return (int)cudaErrorInvalidValue;
+  const long most = (long)(sms > 0 ? sms : 148) * 16;
+  LL_DISPATCH_DTYPE(dtype, {
+    constexpr int VEC = 16 / (int)sizeof(T);
+    const bool wide = shared_ff % VEC == 0 && ff % VEC == 0 && ((uintptr_t)in % 16) == 0 && ((uintptr_t)out % 16) == 0;
+    const long want = (num_tokens * width / (wide ? VEC : 1) + 255) / 256;
+    const dim3 grid((int)(want < most ? want : most));
+    if (wide)
+      ll_launch(moe_gated_act_kernel<T, VEC>, grid, dim3(256), 0, stream, (T*)out, (const T*)in, gates, shared_w,
+                num_tokens, shared_ff, ff, E, limit, shared_limit, alpha);
+    else
+      ll_launch(moe_gated_act_kernel<T, 1>, grid, dim3(256), 0, stream, (T*)out, (const T*)in, gates, shared_w,
+                num_tokens, shared_ff, ff, E, limit, shared_limit, alpha);
+  });
   return LL_LAUNCH_RESULT();
 }
 

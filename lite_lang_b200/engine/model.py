@@ -39,6 +39,7 @@ class PlannedStep:
 
     layer: int
     caches: Dict[str, PlannedCache]
+    add_embedding: bool = False
 
     def _first(self) -> PlannedCache:
         return next(iter(self.caches.values())) if self.caches else PlannedCache(None, 0, False)
@@ -122,7 +123,7 @@ class CausalLM:
                     g = len(keys) - 1
                 caches[role] = PlannedCache(g, planes[g], True)
                 planes[g] += 1
-            plan.append(PlannedStep(rs.layer, caches))
+            plan.append(PlannedStep(rs.layer, caches, rs.add_embedding))
         groups: List[object] = []
         for need, n in zip(keys, planes):
             if isinstance(need, PagedKVNeed):
@@ -197,7 +198,12 @@ class CausalLM:
         n = step.num_tokens
         h = self.embedding.forward(step.token_ids, n, step.status)
         delta = None
+        h0 = h if any(ps.add_embedding for ps in self.plan) else None
+        if h0 is not None and not all(b.keeps_residual for b in self.blocks):
+            h = h0.clone()
         for ps in self.plan:
+            if ps.add_embedding:
+                delta = parts_base.with_extra(delta, h0.float())
             caches = {}
             for role, pc in ps.caches.items():
                 if pc.group is None:

@@ -16,7 +16,7 @@ from __future__ import annotations
 import ctypes
 import os
 from ctypes import c_float, c_int, c_long, c_void_p
-from typing import Optional, Tuple
+from typing import NamedTuple, Optional, Tuple
 
 import torch
 
@@ -251,17 +251,33 @@ def bias_rotate_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], positions
                 _ptr(v_cache), c_int(page_size), c_long(num_slots), c_int(qkv.shape[0]), _ptr(status), _stream())
 
 
-GATE_ACT = {"silu": 0, "relu": 1}
+GATE_ACT = {"silu": 0, "relu": 1, "clamped_swish": 2}
 
 
-def act_mul(out: torch.Tensor, gate_up: torch.Tensor, act: str) -> None:
-    """out = act(gate) * up for the fused projection [tokens, 2 * I] (gate columns first); act silu or relu."""
+class GateAct(NamedTuple):
+    """The activation of a gated product: act(gate) * up with SiLU or ReLU; "clamped_swish": with a = min(gate, limit)
+    and c = clamp(up, -limit, limit), a * sigmoid(alpha a) * (c + 1)."""
+    kind: str
+    limit: float = 0.0
+    alpha: float = 0.0
+
+
+def _gate_act(act) -> GateAct:
+    act = GateAct(act) if isinstance(act, str) else act
+    _need(act.kind in GATE_ACT and (act.kind != "clamped_swish" or act.limit > 0),
+          f"gate activation {act.kind!r}: one of {', '.join(GATE_ACT)} (clamped_swish with a positive limit)")
+    return act
+
+
+def act_mul(out: torch.Tensor, gate_up: torch.Tensor, act) -> None:
+    """out = the gated activation (a name or a ``GateAct``) of the fused projection [tokens, 2 * I], gate columns first."""
     _need_cuda(out, gate_up)
+    act = _gate_act(act)
     _need(gate_up.is_contiguous() and out.is_contiguous() and out.dtype == gate_up.dtype, "act_mul: layout")
     n, two_i = gate_up.shape
     _need(two_i % 2 == 0 and out.shape[0] == n and out.shape[1] == two_i // 2, "act_mul: shapes")
     core().call("ll_act_mul", c_int(_dtype_code(out)), _ptr(out), _ptr(gate_up), c_int(n), c_int(two_i // 2),
-                c_int(GATE_ACT[act]), _stream())
+                c_int(GATE_ACT[act.kind]), c_float(act.limit), c_float(act.alpha), _stream())
 
 
 def add_bias(x: torch.Tensor, bias: torch.Tensor) -> None:
@@ -603,13 +619,14 @@ def smallm_supported(x: torch.Tensor, weight: torch.Tensor) -> bool:
 
 
 def gemm_smallm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated: bool = False,
-                act: str = "silu") -> torch.Tensor:
+                act="silu") -> torch.Tensor:
     """out = x @ weight.T for up to 64 tokens with the weight-streaming kernel.
 
     ``gated``: weight holds gate rows then up rows ([2 I, K]); out [M, I] = silu(gate) * up.
     out may be bfloat16 or (not gated) float32.
     """
     _need_cuda(x, weight, out)
+    act = _gate_act(act)
     _need(smallm_supported(x, weight), "gemm_smallm: bfloat16, at most 64 tokens, K a multiple of 32")
     m, k = x.shape
     n = weight.shape[0] // 2 if gated else weight.shape[0]
@@ -619,8 +636,8 @@ def gemm_smallm(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated:
           "gemm_smallm: out dtype")
     load_library("gemm_smallm").call(
         "ll_gemm_smallm", _ptr(out), c_long(out.stride(0)), c_int(1 if out.dtype == torch.float32 else 0), _ptr(x),
-        c_long(x.stride(0)), _ptr(weight), c_int(m), c_int(n), c_int(k), c_int(1 + GATE_ACT[act] if gated else 0),
-        _stream())
+        c_long(x.stride(0)), _ptr(weight), c_int(m), c_int(n), c_int(k), c_int(1 + GATE_ACT[act.kind] if gated else 0),
+        c_float(act.limit), c_float(act.alpha), _stream())
     return out
 
 
@@ -676,7 +693,7 @@ def stream_ksplit(n: int, k: int, mode: int, device) -> int:
 
 
 def gemm_stream(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, mode: int,
-                status: Optional[torch.Tensor] = None, act: str = "silu", row_act: Optional[str] = None) -> torch.Tensor:
+                status: Optional[torch.Tensor] = None, act="silu", row_act: Optional[str] = None) -> torch.Tensor:
     """out = x @ weight.T for up to 32 bfloat16 tokens (64 for mode 2 to bfloat16 with k whole) with the TMA
     weight-streaming kernel.
 
@@ -687,6 +704,7 @@ def gemm_stream(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, mode: 
     """
     _need_cuda(x, weight, out, status)
     m, k = x.shape
+    act = _gate_act(act)
     gated = mode == 1
     row_code = 0
     if row_act is not None:
@@ -709,8 +727,9 @@ def gemm_stream(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, mode: 
     _need(out.dtype == torch.bfloat16 or (out.dtype == torch.float32 and not gated), "gemm_stream: out dtype")
     load_library("gemm_stream").call(
         "ll_gemm_stream", _ptr(out), c_long(out_stride), c_int(1 if out.dtype == torch.float32 else 0), _ptr(x),
-        c_long(x.stride(0)), _ptr(weight), c_int(m), c_int(n), c_int(k), c_int(mode | (GATE_ACT[act] << 8) | (row_code << 16)),
-        c_int(ksplit), c_int(sm_count(x.device)), _ptr(status if status is not None else TIMELINE_STATUS), _stream())
+        c_long(x.stride(0)), _ptr(weight), c_int(m), c_int(n), c_int(k), c_int(mode | (GATE_ACT[act.kind] << 8) | (row_code << 16)),
+        c_int(ksplit), c_int(sm_count(x.device)), c_float(act.limit), c_float(act.alpha),
+        _ptr(status if status is not None else TIMELINE_STATUS), _stream())
     return out
 
 
@@ -866,12 +885,13 @@ def tc_ksplit(n: int, k: int, device) -> int:
     return (boxes + per - 1) // per
 
 
-def gemm_tc(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated: bool = False, act: str = "silu",
+def gemm_tc(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated: bool = False, act="silu",
             status: Optional[torch.Tensor] = None, sumsq: Optional[torch.Tensor] = None, eps: float = 0.0) -> torch.Tensor:
     """out = x @ weight.T for up to 128 bfloat16 tokens on the tcgen05 tensor cores (weights streamed
     by TMA, accumulator in tensor memory).  ``gated``: weight is [2 I, K] and out = silu(gate) * up.
     A float32 ``out`` of shape [parts, M, N] receives the partial sums of a k range cut into parts."""
     _need_cuda(x, weight, out, status)
+    act = _gate_act(act)
     _need(tc_supported(x, weight), "gemm_tc: bfloat16, at most 128 tokens, K % 64 == 0, 16-byte aligned rows")
     m, k = x.shape
     n = weight.shape[0] // 2 if gated else weight.shape[0]
@@ -889,9 +909,10 @@ def gemm_tc(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated: boo
     _need(out.dtype == torch.bfloat16 or (out.dtype == torch.float32 and not gated), "gemm_tc: out dtype")
     load_library("gemm_tc").call(
         "ll_gemm_tc", _ptr(out), c_long(out_stride), c_int(1 if out.dtype == torch.float32 else 0), _ptr(x),
-        c_long(x.stride(0)), _ptr(weight), c_int(m), c_int(n), c_int(k), c_int(1 + GATE_ACT[act] if gated else 0),
+        c_long(x.stride(0)), _ptr(weight), c_int(m), c_int(n), c_int(k), c_int(1 + GATE_ACT[act.kind] if gated else 0),
         c_int(ksplit),
         c_int(sm_count(x.device)), _ptr(sumsq), c_int(0 if sumsq is None else sumsq.shape[0]), c_float(eps),
+        c_float(act.limit), c_float(act.alpha),
         _ptr(status if status is not None else TIMELINE_STATUS), _stream())
     return out
 
@@ -909,11 +930,12 @@ def pair_supported(x: torch.Tensor, weight: torch.Tensor) -> bool:
 
 
 def gemm_pair(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated: bool = False,
-              status: Optional[torch.Tensor] = None, act: str = "silu", row_act: Optional[str] = None) -> torch.Tensor:
+              status: Optional[torch.Tensor] = None, act="silu", row_act: Optional[str] = None) -> torch.Tensor:
     """out = x @ weight.T for many bfloat16 tokens on the tcgen05 tensor cores, a pair of SMs a tile of
     256 tokens x 256 columns.  ``gated``: weight is [2 I, K] and out = silu(gate) * up, the activation done
     on the accumulator, so gate and up never go to memory."""
     _need_cuda(x, weight, out, status)
+    act = _gate_act(act)
     _need(pair_supported(x, weight), "gemm_pair: bfloat16, K % 8 == 0, 16-byte aligned rows")
     m, k = x.shape
     n = weight.shape[0] // 2 if gated else weight.shape[0]
@@ -927,8 +949,8 @@ def gemm_pair(x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, gated: b
         return out
     load_library("gemm_pair").call(
         "ll_gemm_pair", _ptr(out), c_long(out.stride(0)), _ptr(x), c_long(x.stride(0)), _ptr(weight), c_int(m),
-        c_int(n), c_int(k), c_int(1 + GATE_ACT[act] if gated else 0), c_int(sm_count(x.device)), _ptr(status),
-        _stream())
+        c_int(n), c_int(k), c_int(1 + GATE_ACT[act.kind] if gated else 0), c_int(sm_count(x.device)), c_float(act.limit),
+        c_float(act.alpha), _ptr(status), _stream())
     return out
 
 
@@ -998,8 +1020,10 @@ def linear_accumulate(x: torch.Tensor, weight: torch.Tensor, acc: torch.Tensor) 
     torch.addmm(acc, x, weight.t(), out=acc)
 
 
-def gated_linear(x: torch.Tensor, w_gate_up: torch.Tensor, activation: str = "silu") -> torch.Tensor:
-    """act(x @ Wg.T) * (x @ Wu.T) with W = [Wg; Wu], act SiLU or ReLU: fused for few tokens, else product + kernel."""
+def gated_linear(x: torch.Tensor, w_gate_up: torch.Tensor, activation="silu") -> torch.Tensor:
+    """act(x @ Wg.T) * (x @ Wu.T) with W = [Wg; Wu], act SiLU or ReLU (or another gated activation, see ``GateAct``): in
+    the product's epilogue where a kernel of this package makes the product, else product + kernel."""
+    activation = _gate_act(activation)
     inter = w_gate_up.shape[0] // 2
     act = torch.empty((x.shape[0], inter), dtype=x.dtype, device=x.device)
     if tc_preferred(x, w_gate_up, gated=True):
@@ -1011,7 +1035,7 @@ def gated_linear(x: torch.Tensor, w_gate_up: torch.Tensor, activation: str = "si
     if TC_ENABLED and x.shape[0] >= PAIR_MIN_M and pair_supported(x, w_gate_up):
         return gemm_pair(x, w_gate_up, act, gated=True, act=activation)
     gu = linear(x, w_gate_up)
-    if activation == "silu":
+    if activation.kind == "silu":
         silu_mul(act, gu)
     else:
         act_mul(act, gu, activation)
@@ -1175,11 +1199,12 @@ def delta_out(out: torch.Tensor, o: torch.Tensor, weight: torch.Tensor, gate: to
 def latent_prepare(proj: torch.Tensor, q_off: int, kv_off: int, norm_w: torch.Tensor, eps: float, freq: torch.Tensor,
                    rot_dims: int, positions: torch.Tensor, slot_map: Optional[torch.Tensor], cache: torch.Tensor,
                    q_full: torch.Tensor, H: int, d: int, r: int, R: int, status: Optional[torch.Tensor],
-                   amplitude: float = 1.0, q: Optional[torch.Tensor] = None) -> None:
+                   amplitude: float = 1.0, q: Optional[torch.Tensor] = None, half_split: bool = False) -> None:
     """Per token: the latent's RMS norm and the rotated key part into the cache row, and every head's rotated
     query part into ``q_full`` [tokens, H, R + r] behind the R latent-space numbers (which a product fills).
     ``q``: the rows that hold the query heads at ``q_off`` when they are not rows of ``proj`` (queries made by a
-    second product); ``amplitude``: a factor on cos and sin."""
+    second product); ``amplitude``: a factor on cos and sin; ``half_split``: pairs (i, i + rot_dims / 2) instead of
+    neighbours."""
     _need_cuda(proj, norm_w, freq, positions, slot_map, cache, q_full, q)
     q = proj if q is None else q
     _need(q.dtype == proj.dtype and q.stride(1) == 1 and q.shape[0] == proj.shape[0], "latent_prepare: q rows")
@@ -1195,7 +1220,7 @@ def latent_prepare(proj: torch.Tensor, q_off: int, kv_off: int, norm_w: torch.Te
         "ll_latent_prepare", c_int(_dtype_code(proj)), _ptr(proj), c_long(proj.stride(0)), c_int(q_off), c_int(kv_off),
         _ptr(norm_w), c_float(eps), _ptr(freq), c_int(rot_dims), _ptr(positions), _ptr(slot_map), _ptr(cache),
         c_long(cache.shape[0] * cache.shape[2]), _ptr(q_full), c_int(proj.shape[0]), c_int(H), c_int(d), c_int(r),
-        c_int(R), _ptr(status), c_float(amplitude), _ptr(q), c_long(q.stride(0)), _stream())
+        c_int(R), _ptr(status), c_float(amplitude), _ptr(q), c_long(q.stride(0)), c_int(1 if half_split else 0), _stream())
 
 
 def latent_attention(out: torch.Tensor, q_full: torch.Tensor, cache: torch.Tensor, block_table: torch.Tensor, step,
@@ -1295,35 +1320,51 @@ MOE_ACT_WEIGHT_IN = 16     # added to an activation's code: the expert's weight 
 
 def moe_router(x: torch.Tensor, w_router: torch.Tensor, gates: torch.Tensor, top_idx: torch.Tensor,
                top_w: torch.Tensor, top: int, score: str = "softmax", renormalize: bool = False,
-               bias: Optional[torch.Tensor] = None, shared_w: Optional[torch.Tensor] = None) -> None:
+               bias: Optional[torch.Tensor] = None, shared_w: Optional[torch.Tensor] = None,
+               choice_bias: Optional[torch.Tensor] = None, groups: Tuple[int, int] = (1, 1), weight_scale: float = 1.0,
+               identity_w: Optional[torch.Tensor] = None) -> None:
     """Scores over the experts in float32 and the ``top`` largest: ``gates`` float32 [tokens, E] (zero where an
-    expert was not chosen), ``top_idx`` int32 and ``top_w`` float32 [tokens, top].  ``score`` "softmax_top": the
-    largest logits are chosen and weighted by the softmax over the chosen ones.  ``bias`` float32 [E] is added to
-    the logits.  With ``shared_w`` float32 [tokens], ``w_router`` has one more row and shared_w = sigmoid of it."""
-    _need_cuda(x, w_router, gates, top_idx, top_w, bias, shared_w)
+    expert was not chosen), ``top_idx`` int32 (-1: nothing left to choose) and ``top_w`` float32 [tokens, top].  ``score``
+    "softmax_top": the largest logits are chosen and weighted by the softmax over the chosen ones.  ``bias`` float32 [E]
+    is added to the logits.  With ``shared_w`` float32 [tokens], ``w_router`` has one more row and shared_w = sigmoid of it.
+    ``choice_bias`` float32 [outputs] is added to the scores for the choice only, not in the weights.  ``groups`` (count,
+    keep): the outputs form ``count`` equal groups of neighbours, and only those of the ``keep`` groups with the largest
+    best choice score can be chosen.  ``weight_scale``: a constant on the weights.  ``identity_w`` float32 [tokens]: the
+    router's outputs beyond ``gates``' columns stand for the token's row itself; it receives the sum of their weights."""
+    _need_cuda(x, w_router, gates, top_idx, top_w, bias, shared_w, choice_bias, identity_w)
     _f32(bias, "router bias")
     _f32(shared_w, "shared_w")
     _f32(w_router, "router weight")
     _f32(gates, "gates")
     _f32(top_w, "top_w")
+    _f32(choice_bias, "choice_bias")
+    _f32(identity_w, "identity_w")
     _i32(top_idx, "top_idx")
-    E, hidden = w_router.shape
+    outputs, hidden = w_router.shape
     if shared_w is not None:
-        E -= 1
-    _need(E == gates.shape[1] and (bias is None or bias.numel() == E), "moe_router: experts")
-    _need(E <= 256, f"moe_router: {E} experts are more than the kernel takes (256)")
+        outputs -= 1
+    E = gates.shape[1]
+    _need((outputs == E or (outputs > E and identity_w is not None)) and (bias is None or bias.numel() == outputs)
+          and (choice_bias is None or choice_bias.numel() == outputs), "moe_router: experts")
+    _need(outputs <= 256, f"moe_router: {outputs} experts are more than the kernel takes (256)")
+    count, keep = int(groups[0]), int(groups[1])
+    _need(count >= 1 and outputs % count == 0 and 1 <= keep <= count, "moe_router: equal groups, some of them kept")
+    _need(score != "softmax_top" or (choice_bias is None and count == 1 and identity_w is None and weight_scale == 1.0),
+          "moe_router: softmax_top goes without a choice bias, groups, identities and a scale")
     _need(x.stride(1) == 1 and x.shape[1] == hidden, "moe_router: x rows")
     load_library("moe").call(
         "ll_moe_router", c_int(_dtype_code(x)), _ptr(x), c_long(x.stride(0)), _ptr(w_router), _ptr(bias), _ptr(gates),
-        _ptr(top_idx), _ptr(top_w), _ptr(shared_w), c_int(x.shape[0]), c_int(hidden), c_int(E), c_int(top),
-        c_int(MOE_SCORE[score]), c_int(1 if renormalize else 0), _stream())
+        _ptr(top_idx), _ptr(top_w), _ptr(shared_w), c_int(x.shape[0]), c_int(hidden), c_int(outputs), c_int(top),
+        c_int(MOE_SCORE[score]), c_int(1 if renormalize else 0), _ptr(choice_bias), c_int(count), c_int(keep),
+        c_float(weight_scale), _ptr(identity_w), c_int(E), _stream())
 
 
 def moe_gated_act(h: torch.Tensor, gates: torch.Tensor, shared_w: Optional[torch.Tensor], shared_ff: int, ff: int,
                   E: int, limit: float, shared_limit: float, alpha: float) -> torch.Tensor:
     """[tokens, shared_ff + E * ff] from the first product over all experts' gate and up rows
     [tokens, 2 * (shared_ff + E * ff)]: a * sigmoid(alpha a) * (c + 1) with a = min(gate, limit),
-    c = clamp(up, -limit, limit), times the expert's weight for the token (``shared_w`` for the always-on one)."""
+    c = clamp(up, -limit, limit), or with a limit of 0 silu(gate) * up, times the expert's weight for the token
+    (``shared_w`` for the always-on one)."""
     _need_cuda(h, gates, shared_w)
     _f32(gates, "gates")
     _f32(shared_w, "shared_w")
@@ -1337,7 +1378,8 @@ def moe_gated_act(h: torch.Tensor, gates: torch.Tensor, shared_w: Optional[torch
 
 
 def moe_row_gated_act(h: torch.Tensor, row_w: Optional[torch.Tensor], limit: float, alpha: float) -> torch.Tensor:
-    """[rows, ff] from [rows, 2 * ff] (gate columns, then up columns): the gated activation times the row's weight."""
+    """[rows, ff] from [rows, 2 * ff] (gate columns, then up columns): the gated activation (of ``moe_gated_act``) times
+    the row's weight."""
     _need_cuda(h, row_w)
     _f32(row_w, "row_w")
     _need(h.is_contiguous() and h.shape[1] % 2 == 0 and (row_w is None or row_w.numel() == h.shape[0]),
@@ -1751,19 +1793,23 @@ def attn_shaped(out: torch.Tensor, q: torch.Tensor, q_stride: int, mixed: bool, 
                 sink_values: Optional[torch.Tensor] = None, distance_bias: Optional[torch.Tensor] = None,
                 keep_first: int = 0, softcap: Optional[float] = None,
                 query_temperature: Optional[Tuple[float, int]] = None, gate_channels: bool = False,
-                out_scale: float = 1.0) -> None:
+                out_scale: float = 1.0,
+                distance_slope: Optional[torch.Tensor] = None) -> None:
     """Tensor-core paged attention (bfloat16) with shaped scores: the mechanisms of ``attention_modulated`` for
     head sizes 64 and 128.  ``q``: the projection's rows (head h at h * head_dim), or with ``mixed`` the wider
     queries that ``qkv_norm_rotate_store`` leaves for mixed heads (then ``temperature`` is inside them).
     ``nsplit`` > 1 (every entry brings one token): the keys of a row are cut into parts of ``span`` stages of 64
     keys, each a CTA, joined by a second kernel; nsplit * span must cover the stages any token sees (kept first
     tokens' stages before the window's are walked by the first part besides).  ``sink_values``, ``distance_bias``,
-    ``keep_first``, ``softcap``, ``query_temperature``, ``gate_channels`` and ``out_scale`` are those of
-    ``attention_modulated``.  Launches one kernel, two with ``nsplit`` > 1."""
+    ``keep_first``, ``softcap``, ``query_temperature``, ``gate_channels``, ``out_scale`` and ``distance_slope`` are those
+    of ``attention_modulated``.  Launches one kernel, two with ``nsplit`` > 1."""
     _need_cuda(out, q, gate, temperature, k_cache, v_cache, block_table, cu_q, ctx_len, req_slot, sink_values,
                distance_bias)
+    _need_cuda(distance_slope)
     _f32(sink_values, "sink_values")
     _f32(distance_bias, "distance_bias")
+    _f32(distance_slope, "distance_slope")
+    _need(distance_slope is None or distance_slope.numel() == num_heads, "distance_slope: a number a head")
     _need(sink_values is None or (sink and sink_values.numel() == num_heads), "sink_values: a number a head")
     _need(distance_bias is None or (distance_bias.dim() == 2 and distance_bias.shape[1] == num_heads
                                     and distance_bias.is_contiguous()), "distance_bias is [distances, heads]")
@@ -1801,7 +1847,7 @@ def attn_shaped(out: torch.Tensor, q: torch.Tensor, q_stride: int, mixed: bool, 
         _ptr(status), _ptr(sink_values), _ptr(distance_bias),
         c_int(0 if distance_bias is None else distance_bias.shape[0]), c_int(int(keep_first or 0)),
         c_float(float(softcap or 0.0)), c_float(qt_coef), c_int(qt_every), c_int(1 if gate_channels else 0),
-        c_float(out_scale), _stream())
+        c_float(out_scale), _ptr(distance_slope), _stream())
 
 
 def attention_modulated(out: torch.Tensor, q: torch.Tensor, q_stride: int, gate: Optional[torch.Tensor],
@@ -1813,7 +1859,8 @@ def attention_modulated(out: torch.Tensor, q: torch.Tensor, q_stride: int, gate:
                         status: Optional[torch.Tensor], sink_values: Optional[torch.Tensor] = None,
                         distance_bias: Optional[torch.Tensor] = None, keep_first: int = 0,
                         softcap: Optional[float] = None, query_temperature: Optional[Tuple[float, int]] = None,
-                        gate_channels: bool = False, out_scale: float = 1.0) -> None:
+                        gate_channels: bool = False, out_scale: float = 1.0,
+                        distance_slope: Optional[torch.Tensor] = None) -> None:
     """Attention of every new token over its request's cached keys with shaped scores (any sizes, both dtypes):
     a number a head on the scores (``temperature``), the heads' scores mixed by ``head_mix`` [nh, nh], a window
     or chunks (``mask``, ``mask_size``), one more key of score 0 without a value (``sink``), a sigmoid gate a
@@ -1823,11 +1870,15 @@ def attention_modulated(out: torch.Tensor, q: torch.Tensor, q_stride: int, gate:
     window, the request's first positions stay visible.  ``softcap``: s <- cap tanh(s / cap) before the bias.
     ``query_temperature`` (coef, every): the scores of the query at position p times
     1 + coef ln(floor((p + 1) / every) + 1).  ``gate_channels``: ``gate`` is [tokens, nh * vd], a gate a channel.
-    ``out_scale``: a constant on the output, applied before its one rounding."""
+    ``out_scale``: a constant on the output, applied before its one rounding.  ``distance_slope`` float32 [nh]: a key n
+    positions back has slope_h * n taken off its score (after the cap)."""
     _need_cuda(out, q, gate, k_cache, v_cache, block_table, token_req, req_slot, positions, temperature, head_mix,
                sink_values, distance_bias)
+    _need_cuda(distance_slope)
     _f32(sink_values, "sink_values")
     _f32(distance_bias, "distance_bias")
+    _f32(distance_slope, "distance_slope")
+    _need(distance_slope is None or distance_slope.numel() == num_heads, "distance_slope: a number a head")
     _need(sink_values is None or (sink and sink_values.numel() == num_heads), "sink_values: a number a head")
     _need(distance_bias is None or (distance_bias.dim() == 2 and distance_bias.shape[1] == num_heads
                                     and distance_bias.is_contiguous()), "distance_bias is [distances, heads]")
@@ -1858,4 +1909,113 @@ def attention_modulated(out: torch.Tensor, q: torch.Tensor, q_stride: int, gate:
         c_int(0 if distance_bias is None else distance_bias.shape[0]), c_int(int(keep_first or 0)),
         c_float(float(softcap or 0.0)), c_float(qt_coef), c_int(qt_every),
         c_long(0 if gate is None else gate.stride(0)), c_int(1 if gate_channels else 0), c_float(out_scale),
-        _stream())
+        _ptr(distance_slope), _stream())
+
+
+# --------------------------------------------------------------------------
+# short causal convolutions over time, and the norm that one follows
+# --------------------------------------------------------------------------
+def conv_record_floats(taps: int, channels: int) -> int:
+    """float32 numbers of a request's record: two halves of taps - 1 inputs a channel and their two marks."""
+    return (2 * (taps - 1) * channels + 2 + 3) // 4 * 4
+
+
+def _conv_record(state: torch.Tensor, taps: int, channels: int) -> None:
+    _f32(state, "state")
+    _need(state.dim() == 2 and state.shape[1] == conv_record_floats(taps, channels),
+          "a convolution's records are [request slots, conv_record_floats]")
+
+
+def norm_conv(out: torch.Tensor, residual: torch.Tensor, weight: torch.Tensor, eps: float,
+              res_out: Optional[torch.Tensor] = None, delta: Optional[torch.Tensor] = None,
+              rows_in: Optional[torch.Tensor] = None, rows_w: Optional[torch.Tensor] = None,
+              extra: Optional[torch.Tensor] = None, conv_w: Optional[torch.Tensor] = None,
+              state: Optional[torch.Tensor] = None, step=None, write_state: bool = True,
+              rows: Optional[torch.Tensor] = None) -> None:
+    """r = residual (float32) + delta + rows_w * rows_in + extra, kept in ``res_out``; h = r / sqrt(mean(r^2) + eps) *
+    weight; out = h, or with a causal convolution over the request's tokens (``conv_w`` float32 [taps, hidden], records
+    ``state``) out = h + conv(h).  ``delta``: [tokens, hidden] of ``out``'s dtype, or float32 partial sums [parts, tokens,
+    hidden]; ``rows_in`` of ``out``'s dtype with a number a token; ``extra`` float32.  ``rows`` (without a convolution):
+    only these tokens are normed.  ``res_out`` may be ``residual`` itself only without a convolution."""
+    _need_cuda(out, residual, weight, res_out, delta, rows_in, rows_w, extra, conv_w, state, rows)
+    for t, nm in ((residual, "residual"), (weight, "norm weight"), (res_out, "res_out"), (rows_w, "rows_w"),
+                  (extra, "extra"), (conv_w, "conv_w")):
+        _f32(t, nm)
+    _i32(rows, "rows")
+    n_all, W = residual.shape
+    n = n_all if rows is None else rows.numel()
+    _need(out.is_contiguous() and tuple(out.shape) == (n, W) and weight.numel() == W, "norm_conv: out and weight")
+    for t in (res_out, extra, rows_in):
+        _need(t is None or (t.is_contiguous() and tuple(t.shape) == (n_all, W)), "norm_conv: rows are [tokens, hidden]")
+    _need(rows_in is None or (rows_in.dtype == out.dtype and rows_w is not None and rows_w.numel() == n_all),
+          "norm_conv: rows_in go with a number a token")
+    partial, parts, part_stride = None, 0, 0
+    if delta is not None and delta.dim() == 3:
+        _need(delta.dtype == torch.float32 and delta.is_contiguous() and tuple(delta.shape[1:]) == (n_all, W),
+              "norm_conv: partial sums are contiguous float32 [parts, tokens, hidden]")
+        partial, parts, part_stride, delta = delta, delta.shape[0], n_all * W, None
+    elif delta is not None:
+        _need(delta.is_contiguous() and delta.dtype == out.dtype and tuple(delta.shape) == (n_all, W),
+              "norm_conv: delta layout")
+    taps, stride = 0, 0
+    token_req = cu_q = ctx_len = req_slot = None
+    if conv_w is not None:
+        taps = conv_w.shape[0]
+        _need(conv_w.shape[1] == W and rows is None and state is not None and step is not None
+              and (res_out is None or res_out.data_ptr() != residual.data_ptr()), "norm_conv: convolution")
+        _conv_record(state, taps, W)
+        stride = state.stride(0)
+        token_req, cu_q, ctx_len, req_slot = step.token_req, step.cu_q, step.ctx_len, step.req_slot
+    load_library("short_conv").call(
+        "ll_norm_conv", c_int(_dtype_code(out)), _ptr(out), _ptr(res_out), _ptr(residual), _ptr(delta), _ptr(partial),
+        c_int(parts), c_long(part_stride), _ptr(rows_in), _ptr(rows_w if rows_in is not None else None), _ptr(extra),
+        _ptr(weight), c_float(eps), _ptr(conv_w), c_int(taps), _ptr(state if conv_w is not None else None), c_long(stride),
+        c_int(1 if write_state else 0), _ptr(token_req), _ptr(cu_q), _ptr(ctx_len), _ptr(req_slot), _ptr(rows), c_int(n),
+        c_int(W), c_int(sm_count(out.device)), _stream())
+
+
+def short_conv(out: Optional[torch.Tensor], x: torch.Tensor, conv_w: torch.Tensor, state: torch.Tensor, step,
+               add_input: bool = False, write_state: bool = True, store: Optional[tuple] = None) -> None:
+    """Causal convolution over the request's tokens of the first ``conv_w.shape[1]`` numbers of the rows ``x``
+    (``conv_w`` float32 [taps, channels], records ``state``); ``add_input``: plus the row itself.  ``out`` receives the
+    first ``out.shape[1]`` channels.  ``store`` = (slot_map, k_cache, v_cache, page_size, q_width, status): the channels
+    from q_width on are the heads' keys, then their values, and go into the cache plane."""
+    _need_cuda(out, x, conv_w, state)
+    _f32(conv_w, "conv_w")
+    taps, C = conv_w.shape
+    n = x.shape[0]
+    _conv_record(state, taps, C)
+    _need(x.dim() == 2 and x.stride(1) == 1 and x.shape[1] >= C, "short_conv: x rows")
+    out_w, out_stride = 0, 0
+    if out is not None:
+        out_w, out_stride = min(out.shape[1], C), out.stride(0)
+        _need(out.dtype == x.dtype and out.stride(1) == 1 and out.shape[0] == n and out.data_ptr() != x.data_ptr(),
+              "short_conv: out rows (not in place: other tokens read the input)")
+    slot_map = k_cache = v_cache = status = None
+    page_size, q_w, k_w, hd, vd, nkv, num_slots = 1, 0, 0, 0, 0, 0, 0
+    if store is not None:
+        slot_map, k_cache, v_cache, page_size, q_w, status = store
+    if slot_map is not None:
+        _need_cuda(slot_map, k_cache, v_cache)
+        _i32(slot_map, "slot_map")
+        _need(k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == x.dtype == v_cache.dtype
+              and k_cache.shape[2] == page_size == v_cache.shape[2] and k_cache.shape[1] == v_cache.shape[1],
+              "short_conv: cache plane")
+        nkv, hd, vd = k_cache.shape[1], k_cache.shape[3], v_cache.shape[3]
+        k_w, num_slots = nkv * hd, k_cache.shape[0] * page_size
+        _need(q_w + nkv * (hd + vd) == C, "short_conv: channels are queries, keys, values")
+    load_library("short_conv").call(
+        "ll_short_conv", c_int(_dtype_code(x)), _ptr(out), c_long(out_stride), c_int(out_w), _ptr(x), c_long(x.stride(0)),
+        c_int(C), _ptr(conv_w), c_int(taps), c_int(1 if add_input else 0), _ptr(state), c_long(state.stride(0)),
+        c_int(1 if write_state else 0), _ptr(step.token_req), _ptr(step.cu_q), _ptr(step.ctx_len), _ptr(step.req_slot),
+        _ptr(slot_map), _ptr(k_cache), _ptr(v_cache), c_int(q_w), c_int(k_w), c_int(hd), c_int(vd), c_int(nkv),
+        c_int(page_size), c_long(num_slots), _ptr(status), c_int(n), c_int(sm_count(x.device)), _stream())
+
+
+def gate_rows(x: torch.Tensor, gate: torch.Tensor) -> None:
+    """x <- x * sigmoid(gate) in place, element by element (float32 arithmetic, one rounding); ``gate`` rows of any stride."""
+    _need_cuda(x, gate)
+    _need(x.is_contiguous() and gate.dtype == x.dtype and gate.stride(1) == 1 and tuple(gate.shape) == tuple(x.shape),
+          "gate_rows: rows of one shape and dtype")
+    core().call("ll_gate_rows", c_int(_dtype_code(x)), _ptr(x), _ptr(gate), c_long(gate.stride(0)), c_int(x.shape[0]),
+                c_int(x.shape[1]), _stream())

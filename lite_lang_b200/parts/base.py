@@ -124,6 +124,7 @@ class Norm(Part):
         """
         if isinstance(delta, ResidualCopy):
             delta = None
+        delta = settled(delta, residual.dtype)
         if isinstance(delta, (tuple, list)):
             parts = [whole_output(d, residual.dtype).float() for d in delta if d is not None]
             delta = None
@@ -212,6 +213,41 @@ class ResidualCopy(NamedTuple):
     rows: torch.Tensor        # [tokens, hidden] in the engine's dtype
 
 
+class Pending(NamedTuple):
+    """What has not been added to the residual yet, where it is more than one tensor: a sublayer's output ``y``, rows
+    times a number a token (``rows``, ``rows_w``: experts that pass their input on), and float32 rows (``extra``: the
+    embedding's output, which a layer range that runs again starts with).  A norm that reads a float32 residual adds
+    them all in its pass; ``settled`` makes one tensor of them for the others."""
+    y: Optional[torch.Tensor] = None         # [tokens, hidden], or float32 partial sums [parts, tokens, hidden]
+    rows: Optional[torch.Tensor] = None      # [tokens, hidden] in the engine's dtype
+    rows_w: Optional[torch.Tensor] = None    # float32 [tokens]
+    extra: Optional[torch.Tensor] = None     # float32 [tokens, hidden]
+
+
+def with_extra(delta, extra: torch.Tensor) -> Pending:
+    """The pending output ``delta`` and ``extra`` rows besides."""
+    if delta is None or isinstance(delta, ResidualCopy):
+        return Pending(extra=extra)
+    if isinstance(delta, Pending):
+        return delta._replace(extra=extra if delta.extra is None else delta.extra + extra)
+    if isinstance(delta, torch.Tensor):
+        return Pending(y=delta, extra=extra)
+    raise TypeError(f"rows cannot be added to a pending {type(delta).__name__}")
+
+
+def settled(delta, dtype: torch.dtype):
+    """A ``Pending`` as one tensor of ``dtype`` (None if nothing is pending); anything else as it is."""
+    if not isinstance(delta, Pending):
+        return delta
+    total = None if delta.y is None else (delta.y.sum(0) if delta.y.dim() == 3 else delta.y.float())
+    if delta.rows is not None:
+        part = delta.rows.float() * delta.rows_w[:, None]
+        total = part if total is None else total + part
+    if delta.extra is not None:
+        total = delta.extra if total is None else total + delta.extra
+    return None if total is None else total.to(dtype)
+
+
 class Connection(Part):
     """How a sublayer is joined to the residual: what it reads (``read``: float32 weights over the streams) and how
     its output goes back (``write(y)`` gives the pending ``StreamWrite``)."""
@@ -260,6 +296,7 @@ class Mixer(Part):
 
 def whole_output(out: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
     """A part's output as one [tokens, hidden] tensor of ``dtype`` (partial sums added up)."""
+    out = settled(out, dtype)
     if out.dim() == 3:
         return out.sum(0).to(dtype)
     return out
@@ -291,6 +328,8 @@ class Block(Part):
     """
 
     kind_family = "block"
+    # True: ``forward`` never writes into the residual rows it is given (it returns other ones)
+    keeps_residual = False
     roles: Mapping[str, str] = {}      # role -> family ("mixer", "feed_forward", "norm")
 
     def __init__(self, parts: Mapping[str, Part]):

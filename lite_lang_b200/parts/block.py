@@ -48,6 +48,40 @@ class PreNormMixerOnlyBlock(Block):
         return h, self.mixer.forward(x, step, caches["mixer"])
 
 
+class PreNormConvBlock(Block):
+    """The pre-norm arrangement with a short convolution between each norm and its sublayer:
+    h += mixer(C1(norm(h))); h += feed_forward(C2(norm(h))), C(u) = u + conv(u).  The residual sum, the norm and the
+    convolution are one pass, which writes the summed residual to new rows (the convolution reads the rows of tokens
+    that other CTAs sum)."""
+
+    @property
+    def keeps_residual(self):
+        return all(hasattr(self.named[r], "add_conv_forward") for r, family in self.roles.items() if family == "norm")
+
+    roles = {"mixer_norm": "norm", "mixer_conv": "mixer", "mixer": "mixer",
+             "feed_forward_norm": "norm", "feed_forward_conv": "mixer", "feed_forward": "feed_forward"}
+
+    def forward(self, h, delta, step, caches):
+        h, x = self.mixer_conv.after(self.mixer_norm, h, delta, step, caches["mixer_conv"])
+        a = self.mixer.forward(x, step, caches["mixer"])
+        h, x = self.feed_forward_conv.after(self.feed_forward_norm, h, a, step, caches["feed_forward_conv"])
+        return h, self.feed_forward.forward(x, step)
+
+
+class PreNormConvMixerOnlyBlock(Block):
+    """The same for a layer without a feed-forward."""
+
+    @property
+    def keeps_residual(self):
+        return all(hasattr(self.named[r], "add_conv_forward") for r, family in self.roles.items() if family == "norm")
+
+    roles = {"mixer_norm": "norm", "mixer_conv": "mixer", "mixer": "mixer"}
+
+    def forward(self, h, delta, step, caches):
+        h, x = self.mixer_conv.after(self.mixer_norm, h, delta, step, caches["mixer_conv"])
+        return h, self.mixer.forward(x, step, caches["mixer"])
+
+
 class ParallelBlock(Block):
     """Parallel arrangement: with n = norm(h), h += mixer(n) + feed_forward(n).  One norm; both parts read
     its output.  Their outputs are handed on together and added (to each other, then to the residual
@@ -107,6 +141,8 @@ class OutputNormMixerOnlyBlock(OutputNormBlock):
 
 register_part("block", "pre_norm", PreNormBlock)
 register_part("block", "pre_norm_mixer_only", PreNormMixerOnlyBlock)
+register_part("block", "pre_norm_conv", PreNormConvBlock)
+register_part("block", "pre_norm_conv_mixer_only", PreNormConvMixerOnlyBlock)
 register_part("block", "output_norm", OutputNormBlock)
 register_part("block", "output_norm_mixer_only", OutputNormMixerOnlyBlock)
 register_part("block", "parallel", ParallelBlock)

@@ -12,8 +12,8 @@ q_plain . (Uk_h c) = (Uk_h^T q_plain) . c, the queries are taken into the latent
 over heads, attention runs there (keys: the cached rows; values: their first ``kv_rank`` numbers), and a
 second batched product expands each head's weighted sum of latents with Uv_h.
 
-Rotation: interleaved pairs (2i, 2i+1) of the rotated part's first ``rot_dims`` numbers turn by
-position * ``rot_base``^(-2i / rot_dims); the rest passes unchanged.  Angles (float32 position times a
+Rotation: pairs of the rotated part's first ``rot_dims`` numbers (``rot_layout`` "interleaved": 2i with 2i+1;
+"half_split": i with i + rot_dims / 2) turn by position * ``rot_base``^(-2i / rot_dims); the rest passes unchanged.  Angles (float32 position times a
 float32 frequency rounded from float64), the latent's norm, scores and softmax are float32.
 
 Further parameters, for designs that differ:
@@ -22,6 +22,8 @@ Further parameters, for designs that differ:
 ``sink``         every head's softmax has one more key, of the learned score ``sink`` [heads], without a value
 ``rot_scaling``  (``factor``, ``original``, ``fast``, ``slow``) the slow frequencies stretched and an amplitude on
                  cos and sin, as ``rope_computed`` makes them
+``channel_gate`` the heads side by side times sigmoid(W_g x), a gate a channel, x being the input of the projections
+                 (tensor ``g`` [heads * vdim, hidden])
 """
 
 from __future__ import annotations
@@ -54,6 +56,8 @@ class LatentAttention(Mixer):
         self.q_rank = None if p.get("q_rank") is None else int(p["q_rank"])
         self.sink = bool(p.get("sink", False))
         self.rot_scaling = None if not p.get("rot_scaling") else dict(p["rot_scaling"])
+        self.rot_layout = str(p.get("rot_layout", "interleaved"))
+        self.channel_gate = bool(p.get("channel_gate", False))
         if self.rot_dims % 2 or not (0 <= self.rot_dims <= self.r):
             raise ValueError("latent_attention: rot_dims must be even and at most rot_dim")
         if self.R > 512:
@@ -75,6 +79,8 @@ class LatentAttention(Mixer):
             d["uq"] = TensorDecl((self.H * (self.d + self.r), self.q_rank))
         if self.sink:
             d["sink"] = TensorDecl((self.H,), "bias", std=1.0)
+        if self.channel_gate:
+            d["g"] = TensorDecl((self.H * self.dv, h))
         d.update(self._kv_tensors())
         return d
 
@@ -100,6 +106,15 @@ class LatentAttention(Mixer):
         if self.kv_off != q.shape[0]:
             rows.append(torch.zeros((self.kv_off - q.shape[0], self.hidden_size), dtype=dtype, device=q.device))
         rows.append(fetch("dkv").to(dtype))
+        self.gate_off = (self.kv_off + self.R + self.r + 7) // 8 * 8
+        if self.channel_gate:
+            pad = self.gate_off - self.kv_off - self.R - self.r
+            if pad:
+                rows.append(torch.zeros((pad, self.hidden_size), dtype=dtype, device=q.device))
+            rows.append(fetch("g").to(dtype))
+        width = sum(t.shape[0] for t in rows)
+        if self.channel_gate and width % 8:      # (rows of the product start on 16-byte boundaries)
+            rows.append(torch.zeros((8 - width % 8, self.hidden_size), dtype=dtype, device=q.device))
         self.w_in = torch.cat(rows, dim=0).to(device).contiguous()
         self.norm_w = fetch("dkv.norm").to(torch.float32).to(device).contiguous()
         self.w_uk = fetch("uk").to(dtype).to(device).contiguous().view(self.H, self.d, self.R)
@@ -107,8 +122,9 @@ class LatentAttention(Mixer):
         self.w_o = fetch("o").to(dtype).to(device).contiguous()
         # frequencies as the rotary part makes them (float64, the scaling's ramp, rounded once)
         rope = build_part("position", _PartSpec("rope_computed", {
-            "rotary_dim": self.rot_dims, "theta": self.rot_base, "layout": "interleaved",
+            "rotary_dim": self.rot_dims, "theta": self.rot_base, "layout": self.rot_layout,
             "scaling": self.rot_scaling if self.rot_dims else None}))
+        self.half_split = not rope.interleaved
         freq = rope.frequencies()
         self.amplitude = float(rope.amplitude)
         self.freq = (freq.to(torch.float32) if freq.numel() else torch.zeros(1)).to(device).contiguous()
@@ -143,7 +159,7 @@ class LatentAttention(Mixer):
         q_full = torch.empty((n, H, R + r), dtype=x.dtype, device=dev)
         ops.latent_prepare(proj, 0, self.kv_off, self.norm_w, self.eps, self.freq, self.rot_dims, step.positions,
                            cache.slot_map if cache.writable else None, cache.k, q_full, H, d, r, R, step.status,
-                           amplitude=self.amplitude, q=qrows)
+                           amplitude=self.amplitude, q=qrows, half_split=self.half_split)
         # queries into the latent space: a_h = Uk_h^T q_h, written in front of the rotated parts
         q_plain = qrows[:, :H * (d + r)].view(n, H, d + r)[:, :, :d].permute(1, 0, 2)         # [H, n, d]
         ops.batched_heads(q_plain, self.w_uk, out=q_full[:, :, :R].permute(1, 0, 2))            # [H, n, R]
@@ -151,7 +167,9 @@ class LatentAttention(Mixer):
         self.attend(lat, q_full, step, cache)
         heads = torch.empty((n, H * self.dv), dtype=x.dtype, device=dev)
         ops.batched_heads(lat.permute(1, 0, 2), self.w_uv_t, out=heads.view(n, H, self.dv).permute(1, 0, 2))
-        return ops.linear(heads, self.w_o)
+        if self.channel_gate:
+            ops.gate_rows(heads, proj[:, self.gate_off:self.gate_off + H * self.dv])
+        return ops.linear(heads, self.w_o, partial_ok=self.partial_ok)
 
     def _splits(self, n, step, device):
         """How many CTAs share a query's keys (a CTA takes a query's 8 heads, 16 on tensor cores), and how many tiles

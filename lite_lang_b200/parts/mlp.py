@@ -1,4 +1,4 @@
-"""SiLU-gated feed-forward: down(silu(gate(x)) * up(x)), no biases.
+"""SiLU-gated feed-forward: down(silu(gate(x)) * up(x)), no biases (or another gated activation, see ``ops.GateAct``).
 
 ``litelang/models/qwen2/layer/transformer_layer.py:79-83``; gate and up are fused
 into one projection whose first I columns are the gate
@@ -26,7 +26,12 @@ class GatedMLP(FeedForward):
         act = spec.params.get("activation", "silu")
         if act not in ops.GATE_ACT:
             raise ValueError(f"gated_mlp: activation {act!r} is not built ({', '.join(ops.GATE_ACT)})")
+        # "clamped_swish": with a = min(gate x, ``limit``) and c = clamp(up x, -limit, limit), down(a sigmoid(``swish_alpha``
+        # a) (c + 1))
         self.activation = act
+        self.gate_act = ops.GateAct(act, float(spec.params.get("limit") or 0.0), float(spec.params.get("swish_alpha", 1.702)))
+        if act == "clamped_swish" and not self.gate_act.limit > 0:
+            raise ValueError("gated_mlp: clamped_swish takes a positive limit")
         # ``tensor_names``: (gate, up, down) under the prefix, for checkpoints that call them otherwise
         self.names = tuple(spec.params.get("tensor_names") or ("gate_proj.weight", "up_proj.weight",
                                                                "down_proj.weight"))
@@ -64,7 +69,7 @@ class GatedMLP(FeedForward):
         if isinstance(x, NormSplit):    # the norm before this part, left to its first product
             act = ops.gemm_stream_gated_scaled(x.scaled, self.w_gate_up, x.sumsq, x.eps, step.status)
         else:
-            act = ops.gated_linear(x, self.w_gate_up, self.activation)
+            act = ops.gated_linear(x, self.w_gate_up, self.gate_act)
         if residual is not None and ops.accumulate_preferred(act, self.w_down):
             ops.linear_accumulate(act, self.w_down, residual)
             return None

@@ -29,11 +29,17 @@ One part, every mechanism a parameter, so that a design picks the ones it has:
 ``keep_first``        with a window: the request's first ``keep_first`` positions stay visible to every later
                       token (at their true distances); their pages stay with the request
 ``softcap``           the scaled score goes through cap * tanh(s / cap) (before any bias)
+``distance_slopes``   a number a head: a key n positions back has slope_h * n taken off its score, after the cap
+                      (``geometric_slopes`` makes the usual ones)
+``conv``              so many taps: q, k and v each pass a causal convolution over time, a filter a channel without a
+                      bias, directly after the projection (tensors ``q.conv``, ``k.conv``, ``v.conv`` [channels, taps])
 ``query_temperature`` {"coef", "every"}: the query at position p is multiplied by
                       1 + coef * ln(floor((p + 1) / every) + 1)
 
 The cache holds keys rotated and normalised and values normalised, one plane of pages; with a window or chunks
-the pages that no later token can read go back to the pool while the request lives.  Scores, softmax weights,
+the pages that no later token can read go back to the pool while the request lives.  With ``conv`` the mixer has two
+kinds of memory, the pages (``kv``) and a record with the projections of the last tokens (``conv``), and where nothing
+else is done to q, k and v (no bias, norm, rotation or mixing) the convolution's kernel stores k and v itself.  Scores, softmax weights,
 norms and angles are float32 whatever the engine's dtype is.  q | k | v (| gate) are one product.
 
 Kernels: in bfloat16 with head sizes 64 and 128, tensor cores (``attn_shaped``: prompt portions 128 rows a CTA,
@@ -46,17 +52,18 @@ float32 arithmetic (``attention_modulated``).
 from __future__ import annotations
 
 import math
-from typing import Dict, Optional
+from typing import Dict, Optional, Tuple
 
 import torch
 
 from .. import ops
 from ..config.spec import PartSpec
 from .base import Mixer, PagedKVNeed, TensorDecl, build_part, register_part
+from .short_conv import ConvMemory, PagedMemory, filters
 
 _NAMES = {"q": "q", "k": "k", "v": "v", "o": "o", "q_bias": "q.b", "k_bias": "k.b", "v_bias": "v.b",
           "q_norm": "q.norm", "k_norm": "k.norm", "temperature": "temp", "mix": "talk", "gate": "g",
-          "sink": "sink", "distance_bias": "rel"}
+          "sink": "sink", "distance_bias": "rel", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv"}
 
 
 def distance_bucket(n: int, buckets: int, farthest: float) -> int:
@@ -66,6 +73,11 @@ def distance_bucket(n: int, buckets: int, farthest: float) -> int:
     if n < half:
         return n
     return min(buckets - 1, half + int(math.floor(math.log(n / half) / math.log(farthest / half) * (buckets - half))))
+
+
+def geometric_slopes(heads: int, exponent: float = 8.0) -> Tuple[float, ...]:
+    """2^(-exponent (h + 1) / heads) for head h: slopes of a distance penalty from steep to nearly flat."""
+    return tuple(2.0 ** (-exponent * (h + 1) / heads) for h in range(heads))
 
 
 class ModulatedAttention(Mixer):
@@ -93,6 +105,9 @@ class ModulatedAttention(Mixer):
         self.softcap = None if not p.get("softcap") else float(p["softcap"])
         qt = p.get("query_temperature")
         self.query_temperature = None if not qt else (float(qt["coef"]), int(qt["every"]))
+        slopes = p.get("distance_slopes")
+        self.distance_slopes = None if slopes is None else tuple(float(s) for s in slopes)
+        self.conv = int(p.get("conv") or 0)
         self.mask = str(p.get("mask", "causal"))
         size = p.get("mask_size")
         self.mask_size = None if size is None else int(size)
@@ -112,8 +127,16 @@ class ModulatedAttention(Mixer):
             raise ValueError("modulated_attention: distance_bias needs 'max' (the distance of the last bucket) above 1")
         if self.query_temperature is not None and self.query_temperature[1] <= 0:
             raise ValueError("modulated_attention: query_temperature.every must be positive")
-        if self.head_mix and (self.distance_bias is not None or self.softcap is not None or self.sink_learned):
-            raise ValueError("modulated_attention: mixed heads with a distance bias, a cap or a learned sink are not built")
+        if self.head_mix and (self.distance_bias is not None or self.softcap is not None or self.sink_learned
+                              or self.distance_slopes is not None):
+            raise ValueError("modulated_attention: mixed heads with a distance bias or slope, a cap or a learned sink "
+                             "are not built")
+        if self.distance_slopes is not None and len(self.distance_slopes) != self.num_heads:
+            raise ValueError("modulated_attention: distance_slopes are a number a head")
+        if self.conv and self.qkv_bias:
+            raise ValueError("modulated_attention: a convolution of projections with biases is not built")
+        if not (0 <= self.conv <= 64):
+            raise ValueError("modulated_attention: conv is a number of taps, up to 64")
         pos = p.get("position")
         self.position = build_part("position", pos) if pos is not None else None
         if self.position is not None and not getattr(self.position, "computed", False):
@@ -131,7 +154,17 @@ class ModulatedAttention(Mixer):
         self.sink_w = self.bias_by_distance = None
         # mechanisms that the block-a-token kernel and the mma.sync kernel know and the tcgen05 kernel does not
         self.extended = bool(self.sink_learned or self.channel_gate or self.distance_bias is not None
-                             or self.keep_first or self.softcap is not None or self.query_temperature is not None)
+                             or self.keep_first or self.softcap is not None or self.query_temperature is not None
+                             or self.distance_slopes is not None)
+        self.conv_w = self.slopes = None
+        # with a convolution: the two kinds of memory as members of their own
+        self.members = []
+        if self.conv:
+            self.members = [("kv", PagedMemory(self._pages(), self.prefix)),
+                            ("conv", ConvMemory(self.conv, self.gate_offset, self.prefix))]
+
+    def sub_mixers(self):
+        return self.members
 
     def tensors(self) -> Dict[str, TensorDecl]:
         h, nm = self.hidden_size, self.names
@@ -152,6 +185,9 @@ class ModulatedAttention(Mixer):
             d[nm["gate"]] = TensorDecl((self.num_heads, h))
         if self.channel_gate:
             d[nm["gate"]] = TensorDecl((self.o_width, h))
+        if self.conv:
+            for name, width in (("q_conv", self.q_width), ("k_conv", self.k_width), ("v_conv", self.v_width)):
+                d[nm[name]] = TensorDecl((width, self.conv), "bias", std=0.4)
         if self.sink_learned:
             d[nm["sink"]] = TensorDecl((self.num_heads,), "bias", std=1.0)
         if self.distance_bias is not None:
@@ -185,6 +221,10 @@ class ModulatedAttention(Mixer):
             self.mix = f32("mix")
         if self.sink_learned:
             self.sink_w = f32("sink")
+        if self.conv:
+            self.conv_w = filters(torch.cat([fetch(nm[r]) for r in ("q_conv", "k_conv", "v_conv")], dim=0), device)
+        if self.distance_slopes is not None:
+            self.slopes = torch.tensor(self.distance_slopes, dtype=torch.float32, device=device)
         if self.distance_bias is not None:
             table = fetch(nm["distance_bias"]).to(torch.float32)
             if table.dim() != 2 or table.shape[0] < 2:
@@ -200,6 +240,9 @@ class ModulatedAttention(Mixer):
         return self.w_in.numel() * self.w_in.element_size() + self.w_o.numel() * self.w_o.element_size()
 
     def cache_need(self):
+        return None if self.conv else self._pages()
+
+    def _pages(self) -> PagedKVNeed:
         return PagedKVNeed(self.num_kv_heads, self.head_dim,
                            self.mask_size if self.mask == "window" else None,
                            None if self.vdim == self.head_dim else self.vdim,
@@ -207,12 +250,12 @@ class ModulatedAttention(Mixer):
                            self.keep_first if self.mask == "window" else 0)
 
     def kernel_libraries(self):
-        libs = ["core", "attn_mod"]
+        libs = ["core", "attn_mod"] + (["short_conv"] if self.conv else [])
         if self.w_in is not None and self.w_in.dtype == torch.bfloat16:
             libs.extend(["gemm_smallm", "gemm_stream", "gemm_tc"])
             if self.head_dim in (64, 128) and self.vdim in (64, 128):
                 libs.append("attn_shaped")
-                if not self.head_mix and not self.sink and self.vdim == self.head_dim:
+                if not self.head_mix and not self.sink and not self.extended and self.vdim == self.head_dim and self.mask != "chunk":
                     libs.append("attn_tc")
         return libs
 
@@ -239,6 +282,10 @@ class ModulatedAttention(Mixer):
         n = x.shape[0]
         proj = ops.linear(x, self.w_in)                  # q | k | v (| gate inputs)
         pos = self.position
+        gate = self._gate(proj)
+        record = None
+        if self.conv:
+            cache, record = cache["kv"], cache["conv"]
         # bfloat16 with head sizes the tensor-core kernel takes: mixed heads become one wider query a head
         shaped = ops.attn_shaped_supported(
             proj.dtype, self.num_kv_heads, self.head_dim, self.vdim, cache.page_size, proj.stride(0), self.head_mix)
@@ -248,6 +295,19 @@ class ModulatedAttention(Mixer):
                                   device=proj.device)
         # on that path a head's temperature goes onto its query before the query's one rounding
         fold = shaped and self.head_temperature and not self.head_mix
+        if record is not None:
+            # (the channels side by side in a buffer of their own: other tokens read the projections)
+            direct = pos is None and self.qk_norm is None and not self.value_norm and not fold and mixed_q is None
+            conv = torch.empty((n, ((self.q_width if direct else self.gate_offset) + 7) // 8 * 8), dtype=proj.dtype,
+                               device=proj.device)
+            ops.short_conv(conv[:, :self.q_width] if direct else conv, proj, self.conv_w, record.state, step,
+                           write_state=record.writable,
+                           store=(cache.slot_map, cache.k, cache.v, cache.page_size, self.q_width, step.status)
+                           if direct and cache.writable else None)
+            proj = conv
+            if direct:
+                self._attend_any(shaped, attn, proj, None, gate, step, cache, fold, out_scale)
+                return
         ops.qkv_norm_rotate_store(
             proj, self.b_in, step.positions, None if pos is None else pos.freq,
             1.0 if pos is None else pos.amplitude, bool(pos is None or pos.interleaved), self.num_heads,
@@ -255,28 +315,31 @@ class ModulatedAttention(Mixer):
             self.eps, cache.slot_map if cache.writable else None, cache.k, cache.v, cache.page_size, step.status,
             head_mix=self.mix if mixed_q is not None else None,
             mix_temperature=self.temperature if (mixed_q is not None or fold) else None, mixed_q=mixed_q)
+        self._attend_any(shaped, attn, proj, mixed_q, gate, step, cache, fold, out_scale)
+
+    def _attend_any(self, shaped, attn, proj, mixed_q, gate, step, cache, fold, out_scale) -> None:
         if shaped:
-            self.attend_shaped(attn, proj, mixed_q, step, cache, None if fold else self.temperature, out_scale)
+            self.attend_shaped(attn, proj, mixed_q, gate, step, cache, None if fold else self.temperature, out_scale)
         else:
-            self.attend(attn, proj, step, cache, out_scale)
+            self.attend(attn, proj, gate, step, cache, out_scale)
 
     def _gate(self, proj):
         if self.channel_gate:
             return proj[:, self.gate_offset:self.gate_offset + self.o_width]
         return proj[:, self.gate_offset:self.gate_offset + self.num_heads] if self.head_gate else None
 
-    def attend(self, out, proj, step, cache, out_scale: float = 1.0) -> None:
+    def attend(self, out, proj, gate, step, cache, out_scale: float = 1.0) -> None:
         """Any sizes, both dtypes, float32 arithmetic: a block a token."""
-        ops.attention_modulated(out, proj, proj.stride(0), self._gate(proj), cache.k, cache.v, cache.block_table,
+        ops.attention_modulated(out, proj, proj.stride(0), gate, cache.k, cache.v, cache.block_table,
                                 step.token_req, step.req_slot, step.positions, proj.shape[0], self.num_heads,
                                 self.num_kv_heads, self.head_dim, self.vdim, cache.page_size, self.mask,
                                 self.mask_size, self.sink, self.scale, self.temperature, self.mix, step.status,
                                 sink_values=self.sink_w, distance_bias=self.bias_by_distance,
                                 keep_first=self.keep_first, softcap=self.softcap,
                                 query_temperature=self.query_temperature, gate_channels=self.channel_gate,
-                                out_scale=out_scale)
+                                out_scale=out_scale, distance_slope=self.slopes)
 
-    def attend_shaped(self, out, proj, mixed_q, step, cache, temperature, out_scale: float = 1.0) -> None:
+    def attend_shaped(self, out, proj, mixed_q, gate, step, cache, temperature, out_scale: float = 1.0) -> None:
         """Tensor cores.  Single-token entries come first in a step: their keys are cut into parts of one or more
         stages of 64 keys, a CTA each (as many parts as the step's single tokens leave SMs for, so the order of a
         position's sums depends on how many tokens decode together, within rounding); the portions of prompts after
@@ -289,11 +352,11 @@ class ModulatedAttention(Mixer):
         n_rest = step.num_entries - n_single
         tail = (self.num_heads, self.num_kv_heads, self.head_dim, self.vdim, cache.page_size, self.mask,
                 self.mask_size, self.sink, self.scale, step.status)
-        head = (out, q, q.stride(0), mixed_q is not None, self._gate(proj), temperature, cache.k, cache.v,
+        head = (out, q, q.stride(0), mixed_q is not None, gate, temperature, cache.k, cache.v,
                 cache.block_table)
         more = dict(sink_values=self.sink_w, distance_bias=self.bias_by_distance, keep_first=self.keep_first,
                     softcap=self.softcap, query_temperature=self.query_temperature, gate_channels=self.channel_gate,
-                    out_scale=out_scale)
+                    out_scale=out_scale, distance_slope=self.slopes)
         if n_single > 0:
             if self.mask == "causal":
                 stages = (int(step.max_kv_len) + 63) // 64 + 1
@@ -330,7 +393,7 @@ class ModulatedAttention(Mixer):
             ops.attn_prefill_tc(out, proj, proj.stride(0), cache.k, cache.v, cache.block_table, step.cu_q[n_single:],
                                 step.ctx_len[n_single:], step.req_slot[n_single:], n_rest, plan[0], self.num_heads,
                                 self.num_kv_heads, self.head_dim, cache.page_size, window, self.scale, step.status,
-                                nsplit=plan[1], split_len=plan[2], gate=self._gate(proj))
+                                nsplit=plan[1], split_len=plan[2], gate=gate)
         elif n_rest > 0:
             key = ("attn_shaped", group)
             blocks = step.scratch.get(key)

@@ -12,7 +12,7 @@ from typing import Dict, Optional
 import torch
 
 from .. import ops
-from .base import Norm, ResidualCopy, StreamWrite, TensorDecl, register_part, whole_output
+from .base import Norm, Pending, ResidualCopy, StreamWrite, TensorDecl, register_part, settled, whole_output
 
 
 class RMSNorm(Norm):
@@ -38,6 +38,7 @@ class RMSNorm(Norm):
         return out
 
     def add_forward(self, residual, delta, rows=None):
+        delta = settled(delta, residual.dtype)
         n = residual.shape[0] if rows is None else rows.numel()
         out = torch.empty((n, residual.shape[1]), dtype=residual.dtype, device=residual.device)
         ops.add_rmsnorm(out, residual, delta, self.weight, self.eps, rows)
@@ -76,6 +77,7 @@ class LayerNormF32Residual(Norm):
             raise TypeError("layer_norm_f32: the residual stream of this norm is float32")
         if isinstance(delta, ResidualCopy):      # nothing is pending
             delta = None
+        delta = settled(delta, self.out_dtype)
         deltas = [d for d in (delta if isinstance(delta, (tuple, list)) else (delta,)) if d is not None]
         if len(deltas) > 2:
             raise ValueError("layer_norm_f32: at most two pending outputs can be added in the norm")
@@ -86,6 +88,76 @@ class LayerNormF32Residual(Norm):
         out = torch.empty((n, residual.shape[1]), dtype=self.out_dtype, device=residual.device)
         ops.add_layernorm(out, residual, deltas[0], deltas[1], self.weight, self.eps, rows, partial)
         return out
+
+
+class RMSNormF32Residual(Norm):
+    """RMS norm over a residual stream that is kept in float32 whatever the engine's dtype is; its output has the
+    engine's dtype: y = x / sqrt(mean(x^2) + eps) * (``offset`` + w), offset 1 for checkpoints that store the weight
+    around zero.  ``tensor`` is the weight's name under the prefix.
+
+    ``add_forward`` takes what is pending as one tensor or as a ``Pending`` and adds it in float32, in place.
+    ``add_conv_forward`` also runs the causal convolution that reads the norm (``parts/short_conv.py``) in the same pass
+    and returns new residual rows instead of writing into the old ones."""
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.hidden_size = int(spec.params["hidden_size"])
+        self.eps = float(spec.params["eps"])
+        self.offset = float(spec.params.get("offset", 0.0))
+        self.tensor = str(spec.params.get("tensor", "weight"))
+        self.weight: Optional[torch.Tensor] = None
+        self.out_dtype: Optional[torch.dtype] = None
+
+    def tensors(self) -> Dict[str, TensorDecl]:
+        if self.offset == 0.0:
+            return {self.tensor: TensorDecl((self.hidden_size,), "norm")}
+        return {self.tensor: TensorDecl((self.hidden_size,), "norm", std=0.1, mean=1.0 - self.offset)}
+
+    def load(self, fetch, dtype, device) -> None:
+        self.weight = (fetch(self.tensor).to(torch.float32) + self.offset).to(device).contiguous()
+        self.out_dtype = dtype
+
+    def kernel_libraries(self):
+        return ("core", "short_conv")
+
+    def _pending(self, residual, delta) -> Pending:
+        if residual.dtype != torch.float32:
+            raise TypeError("rms_norm_f32: the residual stream of this norm is float32")
+        if delta is None or isinstance(delta, ResidualCopy):
+            return Pending()
+        if isinstance(delta, Pending):
+            p = delta
+        elif isinstance(delta, torch.Tensor):
+            p = Pending(y=delta)
+        else:
+            raise TypeError(f"rms_norm_f32: a pending {type(delta).__name__} is not built")
+        if p.y is not None and p.y.dim() == 2 and p.y.dtype != self.out_dtype:
+            p = p._replace(y=p.y.to(self.out_dtype))
+        return p
+
+    def forward(self, x, out=None):
+        return self.add_forward(x, None)
+
+    def add_forward(self, residual, delta, rows=None):
+        p = self._pending(residual, delta)
+        n = residual.shape[0] if rows is None else rows.numel()
+        out = torch.empty((n, self.hidden_size), dtype=self.out_dtype, device=residual.device)
+        changed = rows is None and any(t is not None for t in p)
+        ops.norm_conv(out, residual, self.weight, self.eps, res_out=residual if changed else None, delta=p.y,
+                      rows_in=p.rows, rows_w=p.rows_w, extra=p.extra, rows=rows)
+        return out
+
+    def add_conv_forward(self, residual, delta, conv_w, record, step):
+        """(new residual rows, h + conv(h)) with h the norm of the new rows."""
+        p = self._pending(residual, delta)
+        out = torch.empty(residual.shape, dtype=self.out_dtype, device=residual.device)
+        new = residual
+        if any(t is not None for t in p):
+            new = torch.empty_like(residual)
+        ops.norm_conv(out, residual, self.weight, self.eps, res_out=None if new is residual else new, delta=p.y,
+                      rows_in=p.rows, rows_w=p.rows_w, extra=p.extra, conv_w=conv_w, state=record.state, step=step,
+                      write_state=record.writable)
+        return new, out
 
 
 class DynamicTanh(Norm):
@@ -134,6 +206,7 @@ class DynamicTanh(Norm):
         if residual.dtype != torch.float32 or residual.shape[1] != self.streams * self.hidden_size:
             raise TypeError("dynamic_tanh: the residual is float32 [tokens, streams * hidden]")
         y = mix = write = None
+        delta = settled(delta, self.out_dtype)
         if isinstance(delta, StreamWrite):
             y, mix, write = delta
         elif delta is not None:
@@ -192,3 +265,4 @@ register_part("norm", "rms_norm", RMSNorm)
 register_part("norm", "layer_norm_out", OutputLayerNorm)
 register_part("norm", "dynamic_tanh", DynamicTanh)
 register_part("norm", "layer_norm_f32", LayerNormF32Residual)
+register_part("norm", "rms_norm_f32", RMSNormF32Residual)

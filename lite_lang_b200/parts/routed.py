@@ -24,6 +24,14 @@ Further parameters, for designs that differ:
 ``gated``         experts have a gate: down(a * sigmoid(``swish_alpha`` a) * (c + 1)) with a = min(gate x, ``limit``)
                   and c = clamp(up x, -limit, limit) (tensors ``e<i>.gate`` beside ``up`` and ``down``); the shared
                   expert has the same form with ``shared_limit``.
+``gate_form``     with ``gated``: "clamped_swish" (as above, the default) or "silu": down(silu(gate x) * (up x)), no limit.
+``correction``    a number an output of the router (tensor ``correction``) added to the scores for the choice only.
+``groups``        (count, keep): the router's outputs form ``count`` equal groups of neighbours, and only the outputs of the
+                  ``keep`` groups with the largest best choice score can be chosen.
+``weight_scale``  a constant on the chosen experts' weights.
+``identity``      so many of the router's outputs, after the experts', stand for the token's row itself: their output is x.
+                  Their weights' sum times x is handed on with the experts' output (``Pending``) and added where the
+                  residual is summed.
 ``score``         "softmax_top": the ``top`` largest logits are chosen, weighted by the softmax over the chosen only.
 ``router_bias``   a bias on the router's logits (tensor ``router.b``).
 ``shared_gate``   the shared expert's output is multiplied by sigmoid(w . x), one number a token (``shared.sg``).
@@ -39,7 +47,7 @@ from typing import Dict
 import torch
 
 from .. import ops
-from .base import FeedForward, TensorDecl, register_part
+from .base import FeedForward, Pending, TensorDecl, register_part
 
 
 class RoutedExperts(FeedForward):
@@ -64,19 +72,37 @@ class RoutedExperts(FeedForward):
         if self.weight_on not in ("output", "input") or (self.gated and self.weight_on == "input"):
             raise ValueError("routed_experts: weight_on is 'output' or (experts without a gate) 'input'")
         self.weight_in = self.weight_on == "input"
-        if self.gated and not (self.limit > 0 and self.shared_limit > 0):
+        self.gate_form = str(p.get("gate_form", "clamped_swish"))
+        if self.gate_form not in ("clamped_swish", "silu"):
+            raise ValueError(f"routed_experts: gate_form {self.gate_form!r}; built: clamped_swish, silu")
+        if self.gate_form == "silu":
+            self.limit = self.shared_limit = 0.0
+        self.identity = int(p.get("identity") or 0)
+        self.correction = bool(p.get("correction", False))
+        groups = p.get("groups") or (1, 1)
+        self.groups = (int(groups[0]), int(groups[1]))
+        self.weight_scale = float(p.get("weight_scale", 1.0))
+        outputs = self.E + self.identity
+        if self.groups[0] < 1 or outputs % self.groups[0] or not (1 <= self.groups[1] <= self.groups[0]):
+            raise ValueError("routed_experts: groups are (count, keep), count divides the router's outputs, keep is 1 to count")
+        if self.groups[1] * (outputs // self.groups[0]) < self.top:
+            raise ValueError("routed_experts: the kept groups have fewer outputs than are chosen")
+        if self.gated and self.gate_form == "clamped_swish" and not (self.limit > 0 and self.shared_limit > 0):
             raise ValueError("routed_experts: gated experts take a positive limit")
         if (not self.gated and self.activation not in ops.MOE_ACT) or self.score not in ops.MOE_SCORE:
             raise ValueError(f"routed_experts: activation {self.activation!r} / score {self.score!r} is not built")
-        if not (0 < self.top <= self.E <= 256):
-            raise ValueError("routed_experts: 0 < top <= experts <= 256")
+        if self.E <= 0 or not (0 < self.top <= outputs <= 256):
+            raise ValueError("routed_experts: 0 < top <= experts (and identities) <= 256")
         self.w_up = None
 
     def tensors(self) -> Dict[str, TensorDecl]:
         h = self.hidden_size
-        d = {"router": TensorDecl((self.E, h), std=0.3)}
+        outputs = self.E + self.identity
+        d = {"router": TensorDecl((outputs, h), std=0.3)}
         if self.router_bias:
-            d["router.b"] = TensorDecl((self.E,), "bias", std=0.3)
+            d["router.b"] = TensorDecl((outputs,), "bias", std=0.3)
+        if self.correction:
+            d["correction"] = TensorDecl((outputs,), "bias", std=0.05)
         names = [f"e{e}" for e in range(self.E)] + (["shared"] if self.shared_ff else [])
         for nm in names:
             ff = self.shared_ff if nm == "shared" else self.ff
@@ -105,6 +131,7 @@ class RoutedExperts(FeedForward):
             router.append(fetch("shared.sg").to(torch.float32).reshape(1, -1))   # one more row: the shared expert's gate
         self.w_router = torch.cat(router, dim=0).to(device).contiguous()
         self.b_router = fetch("router.b").to(torch.float32).to(device).contiguous() if self.router_bias else None
+        self.choice_bias = fetch("correction").to(torch.float32).to(device).contiguous() if self.correction else None
         # views for the grouped way: the experts' up matrices [E, ff, hidden] inside the stacked one; their down
         # matrices [E, hidden, ff] as strided views of the stacked one's columns
         sff, ff, E, h = self.shared_ff, self.ff, self.E, self.hidden_size
@@ -119,7 +146,7 @@ class RoutedExperts(FeedForward):
     def weight_bytes(self) -> int:
         return sum(t.numel() * t.element_size() for t in (self.w_up, self.w_down, self.w_router))
 
-    _shared_w = None
+    _shared_w = _identity_w = None
 
     def kernel_libraries(self):
         libs = ["core", "moe"]
@@ -133,13 +160,19 @@ class RoutedExperts(FeedForward):
         top_idx = torch.empty((n, self.top), dtype=torch.int32, device=dev)
         top_w = torch.empty((n, self.top), dtype=torch.float32, device=dev)
         self._shared_w = torch.empty((n,), dtype=torch.float32, device=dev) if self.shared_gate else None
+        self._identity_w = torch.empty((n,), dtype=torch.float32, device=dev) if self.identity else None
         ops.moe_router(x, self.w_router, gates, top_idx, top_w, self.top, self.score, self.renormalize,
-                       bias=self.b_router, shared_w=self._shared_w)
+                       bias=self.b_router, shared_w=self._shared_w, choice_bias=self.choice_bias, groups=self.groups,
+                       weight_scale=self.weight_scale, identity_w=self._identity_w)
         return gates, top_idx, top_w
 
     GROUPED_MIN_TOKENS = 128
 
     def forward(self, x, step):
+        y = self._experts(x, step)
+        return Pending(y, rows=x, rows_w=self._identity_w) if self.identity else y
+
+    def _experts(self, x, step):
         gates, idx, wts = self.route(x)
         if self.grouped and x.shape[0] >= self.GROUPED_MIN_TOKENS and not getattr(step, "captured", False):
             try:
