@@ -457,7 +457,7 @@ def run_ours(args):
 
 
 # ---------------------------------------------------------------------------------------------------------
-# --compare nevurax / redirax / lenuzen: that design beside Qwen2 at equal layer sizes (random weights)
+# --compare nevurax / redirax / lenuzen / rufisun / tusipel: that design beside Qwen2 at equal layer sizes (random weights)
 # ---------------------------------------------------------------------------------------------------------
 def _nevurax_shape(width, heads, kv_heads, head, inter, vocab, layers, window, experts, top):
     """A Nevurax model whose layers are as large as a Qwen2 layer of the given sizes: the mixers have as many
@@ -534,8 +534,30 @@ def _rufisun_shape(width, heads, kv_heads, head, inter, vocab, layers, window, e
                        for i in range(layers)]}
 
 
+def _tusipel_shape(width, heads, kv_heads, head, inter, vocab, layers, window, experts, top):
+    """A Tusipel model whose layers are as large as a Qwen2 layer of the given sizes.  The layers take turns: the chunked
+    attention with convolved q, k and v and a distance slope a head (same heads, values as wide as keys) and the latent
+    attention with a window and a gate a channel (a latent of four key heads, queries through a latent of 3/4 of the
+    width), chunk and window of ``window`` positions, four taps everywhere.  The first layer's feed-forward is the dense
+    gated one, the others route ``top`` of ``experts`` gated experts and four identities (four groups, three of them kept)
+    with as many *active* weights as the dense one.  No layer runs twice."""
+    moe = {"kind": "moe", "expert": {"ff": inter // top // 64 * 64},
+           "router": {"experts": experts, "identity": 4, "top": top, "groups": {"count": 4, "keep": 3}, "scale": 2.0}}
+    dense = {"kind": "dense", "ff": inter, "limit": 7.0}
+    attention = {"heads": heads, "kv_heads": kv_heads, "dim": head, "vdim": head, "scale": head ** -0.5, "conv": 4,
+                 "mask": {"size": window}}
+    latent = {"heads": heads, "dim": head - 32, "rot_dim": 32, "vdim": head, "kv_rank": 4 * head,
+              "q_rank": 3 * width // 4 // 64 * 64, "scale": head ** -0.5, "mask": {"size": window},
+              "rot": {"base": 1e6, "dims": 32, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    kinds = [("attention", attention), ("latent_attention", latent)]
+    return {"architecture": "Tusipel", "vocab": vocab, "width": width, "embedding": {"scale": width ** 0.5},
+            "norm": {"eps": 1e-6}, "canon": {"taps": 4},
+            "layers": [{"type": kinds[i % 2][0], "mixer": kinds[i % 2][1], "mlp": dense if i % 4 == 0 else moe}
+                       for i in range(layers)]}
+
+
 COMPARE_DESIGNS = {"nevurax": _nevurax_shape, "redirax": _redirax_shape, "lenuzen": _lenuzen_shape,
-                   "rufisun": _rufisun_shape}
+                   "rufisun": _rufisun_shape, "tusipel": _tusipel_shape}
 
 COMPARE_SIZES = {
     # name: (Qwen2 sizes, window of the latent attention, experts, top)
@@ -565,7 +587,7 @@ def _kernel_table(engine, entries_fn, steps=3):
             a[0] += 1
             a[1] += e.device_time
     return [{"kernel": k, "calls": round(n / steps, 1), "us": round(t / steps, 1)}
-            for k, (n, t) in sorted(agg.items(), key=lambda kv: -kv[1][1])][:14]
+            for k, (n, t) in sorted(agg.items(), key=lambda kv: -kv[1][1])][:20]
 
 
 def run_compare(args):
@@ -632,6 +654,9 @@ def run_compare(args):
             torch.cuda.empty_cache()
         if design_name == "rufisun":
             row["config"] = {design_name: {"window": window, "keep_first": 64, "experts": experts, "top": top,
+                                           "expert_ff": nev["layers"][-1]["mlp"]["expert"]["ff"] if layers > 1 else None}}
+        elif design_name == "tusipel":
+            row["config"] = {design_name: {"window": window, "chunk": window, "experts": experts, "identity": 4, "top": top,
                                            "expert_ff": nev["layers"][-1]["mlp"]["expert"]["ff"] if layers > 1 else None}}
         elif design_name == "lenuzen":
             row["config"] = {design_name: {"window": window, "chunk": window, "ff": nev["layers"][-1]["mlp"]["ff"]}}
@@ -747,9 +772,9 @@ def main():
                     help="with --only: the layer sizes of that workload's model instead of Qwen2-1.5B's")
     ap.add_argument("--design-only", action="store_true", dest="design_only",
                     help="with --compare: leave the Qwen2 arm out")
-    ap.add_argument("--against", default="", choices=["", "qwen2", "nevurax", "redirax", "lenuzen"],
+    ap.add_argument("--against", default="", choices=["", "qwen2", "nevurax", "redirax", "lenuzen", "rufisun"],
                     help="with --compare: the arm beside the design (default qwen2)")
-    ap.add_argument("--compare", default="", choices=["", "nevurax", "redirax", "lenuzen", "rufisun"],
+    ap.add_argument("--compare", default="", choices=["", "nevurax", "redirax", "lenuzen", "rufisun", "tusipel"],
                     help="instead of the headline measurement: prefill and decode of a few layers of that design beside "
                          "Qwen2 at equal layer sizes (random weights); --layers (default 4), --size, --kernels go with it")
     ap.add_argument("--size", default="", dest="shape_name", choices=[""] + sorted(COMPARE_SIZES),

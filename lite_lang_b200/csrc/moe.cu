@@ -23,53 +23,82 @@
 // and outputs real .. E - 1 are identities, whose weights add up to identity_w[t].  choice_bias (float32 [E], optional)
 // is added to the scores for the choice.  With `keep` < `count`, only outputs of the `keep` groups (E / count neighbours
 // each) with the largest best choice score can be chosen.  A place that finds nothing left gets top_idx -1 and weight 0.
-// One block per token: its eight warps share out the experts
-// (the token's row waits in shared memory as float32), then the first warp scores and picks.
-#define MOE_ROUTER_THREADS 256
-template <typename T>
-__global__ void __launch_bounds__(MOE_ROUTER_THREADS)
+//
+// A block takes TOK tokens (one, and then a warp an output; or eight in long portions: the router's matrix is then read
+// once for eight tokens); its warps share out the outputs, and then the tokens, whose scores a warp each makes and picks
+// from.  A lane sums its pieces of four numbers of a row (four sums side by side), then the lanes are added up: an order
+// that depends on the sizes only.
+__device__ __forceinline__ float4 moe_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 moe_load4(const bf16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+  const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+template <typename T, int TOK, int THREADS>
+__global__ void __launch_bounds__(THREADS)
 moe_router_kernel(const T* __restrict__ x, long x_stride, const float* __restrict__ Wr, const float* __restrict__ bias,
                   float* __restrict__ gates, int* __restrict__ top_idx, float* __restrict__ top_w,
                   float* __restrict__ shared_w, int num_tokens, int hidden, int E, int top, int score_fn,
                   int renormalize, const float* __restrict__ choice_bias, int count, int keep, float weight_scale,
-                  float* __restrict__ identity_w, int real) {
-  __shared__ float z[MOE_MAX_E + 2];
-  __shared__ float cs[MOE_MAX_E];                        // choice scores
-  __shared__ float gb[MOE_MAX_E];                        // the groups' best
-  extern __shared__ __align__(16) float xrow[];          // the token's row as float32 [hidden]
+                  float* __restrict__ identity_w, int real, int pitch) {
+  extern __shared__ __align__(16) float moe_smem[];      // [TOK]: logits / scores [E + 1], choice scores [E], groups' best
   LL_PDL_TRIGGER();
   LL_PDL_WAIT();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int t = blockIdx.x;
-  const T* xr = x + (size_t)t * x_stride;
-  for (int i = threadIdx.x; i < hidden; i += MOE_ROUTER_THREADS) xrow[i] = to_f32<T>(xr[i]);
-  __syncthreads();
-  const int n_rows = E + (shared_w ? 1 : 0);
-  // a warp a row: a lane sums its pieces of four numbers (four sums side by side), then the lanes are added up:
-  // an order that depends on the sizes only
-  const bool vec = (hidden & 3) == 0;
-  for (int e = warp; e < n_rows; e += MOE_ROUTER_THREADS / 32) {
-    const float* wrow = Wr + (size_t)e * hidden;
-    float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
-    if (vec) {
-#pragma unroll 4
-      for (int i = 4 * lane; i < hidden; i += 128) {
-        const float4 w4 = *reinterpret_cast<const float4*>(wrow + i);
-        const float4 x4 = *reinterpret_cast<const float4*>(xrow + i);
-        a0 = fmaf(w4.x, x4.x, a0);
-        a1 = fmaf(w4.y, x4.y, a1);
-        a2 = fmaf(w4.z, x4.z, a2);
-        a3 = fmaf(w4.w, x4.w, a3);
-      }
-    } else {
-#pragma unroll 4
-      for (int i = lane; i < hidden; i += 32) a0 = fmaf(wrow[i], xrow[i], a0);
+  const int tok0 = blockIdx.x * TOK, nt = min(TOK, num_tokens - tok0);
+  const int zs = 2 * E + 1 + count;
+  T* xrow = reinterpret_cast<T*>(moe_smem + (TOK * zs + 3) / 4 * 4);     // the tokens' rows, `pitch` apart
+  constexpr int VEC = 16 / (int)sizeof(T);
+  if ((hidden % VEC) == 0 && (x_stride % VEC) == 0 && ((uintptr_t)x % 16) == 0) {
+    const int per = hidden / VEC;
+    for (int i = threadIdx.x; i < nt * per; i += THREADS) {
+      const int k = i / per, c = (i - k * per) * VEC;
+      *reinterpret_cast<uint4*>(xrow + (size_t)k * pitch + c) =
+          *reinterpret_cast<const uint4*>(x + (size_t)(tok0 + k) * x_stride + c);
     }
-    const float a = warp_sum((a0 + a1) + (a2 + a3));
-    if (lane == 0) z[e] = a + ((bias && e < E) ? bias[e] : 0.f);
+  } else {
+    for (int k = 0; k < nt; ++k)
+      for (int i = threadIdx.x; i < hidden; i += THREADS) xrow[(size_t)k * pitch + i] = x[(size_t)(tok0 + k) * x_stride + i];
   }
   __syncthreads();
-  if (warp != 0) return;
+  const int n_rows = E + (shared_w ? 1 : 0);
+  const bool vec = (hidden & 3) == 0;
+  for (int e = warp; e < n_rows; e += THREADS / 32) {
+    float a[TOK][4];
+#pragma unroll
+    for (int k = 0; k < TOK; ++k) a[k][0] = a[k][1] = a[k][2] = a[k][3] = 0.f;
+    const float* wrow = Wr + (size_t)e * hidden;
+    if (vec) {
+#pragma unroll(TOK == 1 ? 8 : 4)
+      for (int i = 4 * lane; i < hidden; i += 128) {
+        const float4 w4 = *reinterpret_cast<const float4*>(wrow + i);
+#pragma unroll
+        for (int k = 0; k < TOK; ++k) {
+          const float4 x4 = moe_load4(xrow + (size_t)k * pitch + i);
+          a[k][0] = fmaf(w4.x, x4.x, a[k][0]);
+          a[k][1] = fmaf(w4.y, x4.y, a[k][1]);
+          a[k][2] = fmaf(w4.z, x4.z, a[k][2]);
+          a[k][3] = fmaf(w4.w, x4.w, a[k][3]);
+        }
+      }
+    } else {
+      for (int i = lane; i < hidden; i += 32)
+#pragma unroll
+        for (int k = 0; k < TOK; ++k) a[k][0] = fmaf(wrow[i], to_f32<T>(xrow[(size_t)k * pitch + i]), a[k][0]);
+    }
+#pragma unroll
+    for (int k = 0; k < TOK; ++k) {
+      const float v = warp_sum((a[k][0] + a[k][1]) + (a[k][2] + a[k][3]));
+      if (lane == 0 && k < nt) moe_smem[k * zs + e] = v + ((bias && e < E) ? bias[e] : 0.f);
+    }
+  }
+  __syncthreads();
+  if (warp >= nt) return;                                // (from here on a warp a token)
+  const int t = tok0 + warp;
+  float* z = moe_smem + warp * zs;
+  float* cs = z + E + 1;                                 // choice scores
+  float* gb = cs + E;                                    // the groups' best
   if (shared_w && lane == 0) shared_w[t] = 1.0f / (1.0f + expf(-z[E]));
   if (score_fn == 2) {
     // the logits themselves are compared; the weights are made from the chosen ones below
@@ -233,12 +262,26 @@ extern "C" int ll_moe_router(int dtype, const void* x, long x_stride, const floa
   if (real <= 0 || real > E || (real < E && identity_w == nullptr) || count < 1 || E % count != 0 || keep < 1 || keep > count)
     return (int)cudaErrorInvalidValue;
   if (E <= 0 || E > MOE_MAX_E || top <= 0 || top > E || hidden <= 0) return (int)cudaErrorInvalidValue;
-  const size_t smem = sizeof(float) * (size_t)((hidden + 3) / 4 * 4);
-  if (smem > 40 * 1024) return (int)cudaErrorInvalidValue;      // (rows of up to 10,240 numbers)
-  LL_DISPATCH_DTYPE(dtype, ll_launch(moe_router_kernel<T>, dim3(num_tokens), dim3(MOE_ROUTER_THREADS), smem, stream,
-                                     (const T*)x, x_stride, Wr, bias, gates, top_idx, top_w, shared_w, num_tokens,
-                                     hidden, E, top, score_fn, renormalize, choice_bias, count, keep, weight_scale,
-                                     identity_w, real));
+  const int zs = 2 * E + 1 + count, pitch = (hidden + 7) / 8 * 8;
+#define MOE_ROUTER_LAUNCH(TOK, THREADS)                                                                                  \
+  do {                                                                                                                   \
+    const size_t smem = sizeof(float) * (size_t)((TOK * zs + 3) / 4 * 4) + sizeof(T) * (size_t)TOK * pitch;              \
+    if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;                                                            \
+    if (smem > 48 * 1024)                                                                                                \
+      cudaFuncSetAttribute(moe_router_kernel<T, TOK, THREADS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);  \
+    ll_launch(moe_router_kernel<T, TOK, THREADS>, dim3((num_tokens + TOK - 1) / TOK), dim3(THREADS), smem,               \
+              stream, (const T*)x, x_stride, Wr, bias, gates, top_idx, top_w, shared_w, num_tokens, hidden, E, top,      \
+              score_fn, renormalize, choice_bias, count, keep, weight_scale, identity_w, real, pitch);                   \
+  } while (0)
+  LL_DISPATCH_DTYPE(dtype, {
+    if (num_tokens >= 512 && sizeof(float) * 8 * (size_t)zs + sizeof(T) * 8 * (size_t)pitch <= 100 * 1024)
+      MOE_ROUTER_LAUNCH(8, 256);
+    else if (E > 8)
+      MOE_ROUTER_LAUNCH(1, 1024);
+    else
+      MOE_ROUTER_LAUNCH(1, 256);
+  });
+#undef MOE_ROUTER_LAUNCH
   return LL_LAUNCH_RESULT();
 }
 

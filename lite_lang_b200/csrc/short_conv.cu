@@ -28,6 +28,7 @@ struct ConvRecord {
   const int* cu_q;        // first token of each entry
   const int* ctx_len;     // tokens of the request before this step
   const int* req_slot;    // the request's slot, -1: padding
+  int single;             // every entry brings one token: token t is entry t (two look-ups less in a row)
 };
 
 // What a token has to know of its entry
@@ -37,11 +38,14 @@ struct ConvToken {
 };
 __device__ __forceinline__ ConvToken conv_token(const ConvRecord& c, int t, int halves) {
   ConvToken k;
-  const int e = c.token_req[t];
+  const int e = c.single ? t : c.token_req[t];
   k.slot = e >= 0 ? c.req_slot[e] : -1;
-  k.first = k.slot >= 0 ? c.cu_q[e] : t;
-  k.last = k.slot >= 0 ? c.cu_q[e + 1] - 1 : t;
-  k.ctx = k.slot >= 0 ? c.ctx_len[e] : 0;
+  k.ctx = e >= 0 ? c.ctx_len[e] : 0;
+  k.first = k.last = t;
+  if (!c.single && k.slot >= 0) {
+    k.first = c.cu_q[e];
+    k.last = c.cu_q[e + 1] - 1;
+  }
   k.rd = 0;
   if (k.slot >= 0) {
     const int* tag = reinterpret_cast<const int*>(c.state + (size_t)k.slot * c.stride + halves);
@@ -148,6 +152,7 @@ struct NormConvParams {
   int n, W, C, segs;      // rows of `out`; tokens a CTA; pieces a row's sum is made of
 };
 
+// Any sizes: the rows of a few tokens (and those before them) wait in shared memory between the norm and the convolution.
 template <typename T, int VEC, int TAPS>
 __global__ void __launch_bounds__(512) norm_conv_kernel(const NormConvParams p) {
   constexpr bool CONV = TAPS > 0;
@@ -167,7 +172,7 @@ __global__ void __launch_bounds__(512) norm_conv_kernel(const NormConvParams p) 
   int from = t0;                                    // the first row this CTA needs
   if (CONV) {
     if (tid < nt) tok_s[tid] = conv_token(p.rec, t0 + tid, 2 * hist * W);
-    const int e = p.rec.token_req[t0];
+    const int e = p.rec.single ? -1 : p.rec.token_req[t0];
     from = max(e >= 0 ? p.rec.cu_q[e] : t0, t0 - hist);
   }
   const int vecs = W / VEC, per = (vecs + segs - 1) / segs;
@@ -316,6 +321,162 @@ __global__ void __launch_bounds__(512) norm_conv_kernel(const NormConvParams p) 
   }
 }
 
+// The usual sizes (rows of up to 4,096 numbers, a multiple of four; up to four taps): a CTA walks a run of tokens, a
+// thread keeps its four channels' last inputs, filters and norm weights in registers, and the rows of the next NW_AHEAD
+// tokens are on their way to shared memory by cp.async while a row is summed (a thread reads back what it copied
+// itself, so the copies need no barrier).  A row costs one barrier and is read once, but for the taps - 1 rows before a
+// CTA's first token, which are normed again for the convolution.
+#define NW_MAX_THREADS 1024
+#define NW_AHEAD 4
+
+template <int BYTES> __device__ __forceinline__ void nw_copy(unsigned dst, const void* src) {
+  if constexpr (BYTES == 16)
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+  else
+    asm volatile("cp.async.ca.shared.global [%0], [%1], %2;" ::"r"(dst), "l"(src), "n"(BYTES) : "memory");
+}
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(NW_MAX_THREADS) norm_conv_walk_kernel(const NormConvParams p) {
+  constexpr int HIST = TAPS - 1, TB = 4 * (int)sizeof(T);
+  constexpr int HN = HIST > 0 ? HIST : 1;
+  extern __shared__ __align__(16) float sc_smem[];      // [NW_AHEAD][residual 16 | pending TB | rows TB][threads]
+  __shared__ float red[2][32];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nthreads = blockDim.x, nwarps = nthreads >> 5;
+  const int W = p.W, c = tid * 4;
+  const bool active = c < W;
+  // (the weights do not depend on the kernel before: they are on their way before the wait for it)
+  float w[4] = {0.f, 0.f, 0.f, 0.f}, cw[TAPS][4];
+  if (active) sc_load<float, 4>(w, p.w + c);
+#pragma unroll
+  for (int j = 0; j < TAPS; ++j) {
+    cw[j][0] = cw[j][1] = cw[j][2] = cw[j][3] = 0.f;
+    if (active) sc_load<float, 4>(cw[j], p.conv_w + (size_t)j * W + c);
+  }
+  LL_PDL_TRIGGER();
+  LL_PDL_WAIT();
+  const int t0 = blockIdx.x * p.C, t1 = min(p.n, t0 + p.C);
+  char* const ring = reinterpret_cast<char*>(sc_smem);
+  const int stage = nthreads * (16 + 2 * TB);
+  const int o_res = tid * 16, o_del = nthreads * 16 + tid * TB, o_row = nthreads * (16 + TB) + tid * TB;
+  auto fetch = [&](int t) {                             // one group a token, empty behind the last
+    if (active && t < t1) {
+      const size_t off = (size_t)t * W + c;
+      const unsigned dst = (unsigned)__cvta_generic_to_shared(ring + (t & (NW_AHEAD - 1)) * stage);
+      nw_copy<16>(dst + o_res, p.res + off);
+      if (p.delta) nw_copy<TB>(dst + o_del, reinterpret_cast<const T*>(p.delta) + off);
+      if (p.rows_in) nw_copy<TB>(dst + o_row, reinterpret_cast<const T*>(p.rows_in) + off);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  // rows that no entry of the CTA's first token needs are copied too where that saves a look-up first
+  int from = max(t0 - HIST, 0);
+  if (p.rec.single) from = t0;
+#pragma unroll
+  for (int i = 0; i < NW_AHEAD - 1; ++i) fetch(from + i);
+  ConvToken k = conv_token(p.rec, t0, 2 * HIST * W);
+  const int need = max(k.first, t0 - HIST);
+  float h[HN][4];
+#pragma unroll
+  for (int i = 0; i < HN; ++i) h[i][0] = h[i][1] = h[i][2] = h[i][3] = 0.f;
+  for (int t = from; t < t1; ++t) {
+    fetch(t + NW_AHEAD - 1);
+    asm volatile("cp.async.wait_group %0;" ::"n"(NW_AHEAD - 1) : "memory");
+    if (t < need) continue;                             // (the same for all threads)
+    if (t > k.last) k = conv_token(p.rec, t, 2 * HIST * W);
+    const size_t off = (size_t)t * W + c;
+    float v[4] = {0.f, 0.f, 0.f, 0.f};
+    if (active) {
+      const char* st = ring + (t & (NW_AHEAD - 1)) * stage;
+      float d[4] = {0.f, 0.f, 0.f, 0.f}, x[4];
+      sc_load<float, 4>(v, reinterpret_cast<const float*>(st + o_res));
+      if (p.delta) {
+        sc_load<T, 4>(d, reinterpret_cast<const T*>(st + o_del));
+      } else if (p.partial) {
+        const float* par = p.partial + off;
+#pragma unroll 4
+        for (int s = 0; s < p.parts; ++s) {
+          sc_load<float, 4>(x, par + (size_t)s * p.part_stride);
+#pragma unroll
+          for (int i = 0; i < 4; ++i) d[i] += x[i];
+        }
+      }
+      if (p.rows_in) {
+        sc_load<T, 4>(x, reinterpret_cast<const T*>(st + o_row));
+        const float pw = p.rows_w[t];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) d[i] = fmaf(pw, x[i], d[i]);
+      }
+      if (p.extra) {
+        sc_load<float, 4>(x, p.extra + off);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) d[i] += x[i];
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) v[i] += d[i];
+      if (t >= t0 && p.res_out) sc_store<float, 4>(p.res_out + off, v);
+      if (HIST > 0 && t == k.first) {                   // the inputs of earlier steps (zeros at the request's start);
+        const float* base = p.rec.state + (size_t)max(k.slot, 0) * p.rec.stride + c;   // needed behind the barrier only
+#pragma unroll
+        for (int i = 0; i < HIST; ++i) {
+          h[i][0] = h[i][1] = h[i][2] = h[i][3] = 0.f;
+          if (k.slot >= 0) sc_load<float, 4>(h[i], base + (size_t)(k.rd * HIST + i) * W);
+        }
+      }
+    }
+    const float ss = warp_sum(fmaf(v[0], v[0], v[1] * v[1]) + fmaf(v[2], v[2], v[3] * v[3]));
+    float* slot = red[t & 1];                           // (two sets: a warp may be a row ahead of another's reads)
+    if (lane == 0) slot[warp] = ss;
+    __syncthreads();
+    const float inv = 1.0f / sqrtf(warp_sum(lane < nwarps ? slot[lane] : 0.f) / (float)W + p.eps);
+    if (!active) continue;
+    float now[4], y[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      now[i] = v[i] * inv * w[i];
+      y[i] = now[i];
+    }
+    if (t >= t0) {
+#pragma unroll
+      for (int j = 0; j < HIST; ++j)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) y[i] = fmaf(cw[j][i], h[j][i], y[i]);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) y[i] = fmaf(cw[TAPS - 1][i], now[i], y[i]);
+      sc_store<T, 4>(reinterpret_cast<T*>(p.out) + off, y);
+      if (k.slot >= 0 && p.rec.write) conv_leave<4>(p.rec, k, t, HIST, W, c, now);
+    }
+#pragma unroll
+    for (int j = 0; j + 1 < HIST; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) h[j][i] = h[j + 1][i];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) h[HN - 1][i] = now[i];
+  }
+  asm volatile("cp.async.wait_all;" ::: "memory");
+}
+
+template <typename T, int TAPS>
+static int nw_launch(NormConvParams p, int sms, cudaStream_t stream) {
+  const int threads = (p.W / 4 + 31) / 32 * 32;
+  const int slots = sms * (threads <= 512 ? 2 : 1);     // CTAs that are resident at once
+  p.C = (p.n + slots - 1) / slots;
+  const size_t smem = (size_t)NW_AHEAD * threads * (16 + 8 * sizeof(T));
+  cudaFuncSetAttribute(norm_conv_walk_kernel<T, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  ll_launch(norm_conv_walk_kernel<T, TAPS>, dim3((p.n + p.C - 1) / p.C), dim3(threads), smem, stream, p);
+  return LL_LAUNCH_RESULT();
+}
+
+template <typename T>
+static int nw_taps(const NormConvParams& p, int sms, cudaStream_t stream) {
+  switch (p.taps) {
+    case 1: return nw_launch<T, 1>(p, sms, stream);
+    case 2: return nw_launch<T, 2>(p, sms, stream);
+    case 3: return nw_launch<T, 3>(p, sms, stream);
+    default: return nw_launch<T, 4>(p, sms, stream);
+  }
+}
+
 static size_t nc_smem(int W, int rows, int segs) { return sizeof(float) * ((size_t)rows * W + rows + (size_t)rows * segs); }
 
 template <typename T, int VEC, int TAPS>
@@ -354,7 +515,7 @@ extern "C" int ll_norm_conv(int dtype, void* out, float* res_out, const float* r
                             const float* partial, int parts, long part_stride, const void* rows_in, const float* rows_w,
                             const float* extra, const float* w, float eps, const float* conv_w, int taps, float* state,
                             long state_stride, int write_state, const int* token_req, const int* cu_q,
-                            const int* ctx_len, const int* req_slot, const int* rows, int n, int W, int sms,
+                            const int* ctx_len, const int* req_slot, int single, const int* rows, int n, int W, int sms,
                             cudaStream_t stream) {
   if (n <= 0) return 0;
   if (W <= 0 || sms <= 0 || (conv_w != nullptr && (taps < 1 || taps > 64 || state == nullptr || rows != nullptr || res_out == res)) ||
@@ -375,7 +536,7 @@ extern "C" int ll_norm_conv(int dtype, void* out, float* res_out, const float* r
   p.eps = eps;
   p.conv_w = conv_w;
   p.taps = taps;
-  p.rec = {state, state_stride, write_state, token_req, cu_q, ctx_len, req_slot};
+  p.rec = {state, state_stride, write_state, token_req, cu_q, ctx_len, req_slot, single};
   p.rows = rows;
   p.n = n;
   p.W = W;
@@ -383,6 +544,8 @@ extern "C" int ll_norm_conv(int dtype, void* out, float* res_out, const float* r
   // (all bases come from an allocator that aligns them well; rows of a multiple of four numbers then start on 16-byte
   // boundaries, and 8-byte ones of bfloat16)
   const bool v4 = (W % 4) == 0 && (part_stride % 4) == 0 && (state_stride % 4) == 0;
+  if (v4 && conv_w != nullptr && taps <= 4 && W <= 4 * NW_MAX_THREADS)
+    LL_DISPATCH_DTYPE(dtype, return nw_taps<T>(p, sms, stream));
   LL_DISPATCH_DTYPE(dtype, return v4 ? nc_taps<T, 4>(p, sms, stream) : nc_taps<T, 1>(p, sms, stream));
 }
 
@@ -406,69 +569,103 @@ struct ShortConvParams {
   int q_w, k_w, hd, vd, nkv, page_size;
   long num_slots;
   int* status;
-  int n, per_thread;      // tokens; tokens a thread walks
+  int n;                  // tokens
 };
 
 #define SC_TY 8
-template <typename T, int VEC, int TAPS>
+template <typename T, int VEC> struct ScRaw { T v[VEC]; };
+template <typename T, int VEC> __device__ __forceinline__ void sc_load_raw(ScRaw<T, VEC>& r, const T* p) {
+  if constexpr (VEC * sizeof(T) == 16) *reinterpret_cast<uint4*>(r.v) = *reinterpret_cast<const uint4*>(p);
+  else r.v[0] = p[0];
+}
+
+// A thread works on VEC channels of NT neighbouring tokens: their rows and the taps - 1 before them are asked for at once.
+template <typename T, int VEC, int TAPS, int NT>
 __global__ void __launch_bounds__(32 * SC_TY) short_conv_kernel(const ShortConvParams p) {
-  LL_PDL_TRIGGER();
-  LL_PDL_WAIT();
+  constexpr int HIST = TAPS == SC_ANY ? 0 : TAPS - 1;   // (SC_ANY: older rows are read where they are used)
   const int taps = TAPS == SC_ANY ? p.taps : TAPS;
   const int hist = taps - 1;
   const int c = (blockIdx.x * 32 + threadIdx.x) * VEC;
-  const int ta = (blockIdx.y * SC_TY + threadIdx.y) * p.per_thread, tb = min(p.n, ta + p.per_thread);
-  if (c >= p.C) return;
-  const T* x = reinterpret_cast<const T*>(p.x);
+  const int ta = (blockIdx.y * SC_TY + threadIdx.y) * NT;
+  const bool active = c < p.C && ta < p.n;
   float cw[TAPS == SC_ANY ? 1 : TAPS][VEC];
   if constexpr (TAPS != SC_ANY) {
+    if (active) {
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) sc_load<float, VEC>(cw[j], p.w + (size_t)j * p.C + c);
+      for (int j = 0; j < TAPS; ++j) sc_load<float, VEC>(cw[j], p.w + (size_t)j * p.C + c);
+    }
   }
-  for (int t = ta; t < tb; ++t) {
-    const ConvToken k = conv_token(p.rec, t, 2 * hist * p.C);
+  LL_PDL_TRIGGER();
+  LL_PDL_WAIT();
+  if (!active) return;
+  const T* x = reinterpret_cast<const T*>(p.x) + c;
+  ScRaw<T, VEC> raw[NT + HIST];
+#pragma unroll
+  for (int i = 0; i < NT + HIST; ++i) {
+    const int t = ta - HIST + i;
+    // (a step of single tokens never reads another token's row)
+    if (t >= 0 && t < p.n && !(p.rec.single && i < HIST)) sc_load_raw<T, VEC>(raw[i], x + (size_t)t * p.x_stride);
+    else
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) raw[i].v[k] = from_f32<T>(0.f);
+  }
+  ConvToken k = conv_token(p.rec, ta, 2 * hist * p.C);
+#pragma unroll
+  for (int n = 0; n < NT; ++n) {
+    const int t = ta + n;
+    if (t >= p.n) break;
+    if (t > k.last) k = conv_token(p.rec, t, 2 * hist * p.C);
     float now[VEC], y[VEC];
-    sc_load<T, VEC>(now, x + (size_t)t * p.x_stride + c);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) y[i] = p.add ? now[i] : 0.f;
-    auto tap = [&](int j, const float (&f)[VEC]) {
-      const int d = hist - j;
-      float h[VEC];
-      if (d == 0) {
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) h[i] = now[i];
-      } else if (t - d >= k.first) {
-        sc_load<T, VEC>(h, x + (size_t)(t - d) * p.x_stride + c);
-      } else if (k.slot >= 0) {
-        sc_load<float, VEC>(h, p.rec.state + (size_t)k.slot * p.rec.stride +
-                                   ((size_t)k.rd * hist + (hist + t - k.first - d)) * p.C + c);
-      } else {
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) h[i] = 0.f;
-      }
-#pragma unroll
-      for (int i = 0; i < VEC; ++i) y[i] = fmaf(f[i], h[i], y[i]);
-    };
+    for (int i = 0; i < VEC; ++i) {
+      now[i] = to_f32<T>(raw[n + HIST].v[i]);
+      y[i] = p.add ? now[i] : 0.f;
+    }
+    const float* rec = p.rec.state + (size_t)max(k.slot, 0) * p.rec.stride + (size_t)k.rd * hist * p.C + c;
     if constexpr (TAPS == SC_ANY) {
       for (int j = 0; j < taps; ++j) {
-        float f[VEC];
+        const int d = hist - j;
+        float f[VEC], h[VEC];
         sc_load<float, VEC>(f, p.w + (size_t)j * p.C + c);
-        tap(j, f);
+        if (t - d >= k.first) {
+          sc_load<T, VEC>(h, x + (size_t)(t - d) * p.x_stride);
+        } else if (k.slot >= 0) {
+          sc_load<float, VEC>(h, rec + (size_t)(hist + t - k.first - d) * p.C);
+        } else {
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) h[i] = 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) y[i] = fmaf(f[i], h[i], y[i]);
       }
     } else {
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) tap(j, cw[j]);
+      for (int j = 0; j < TAPS; ++j) {
+        const int d = TAPS - 1 - j;
+        float h[VEC];
+        if (t - d >= k.first) {
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) h[i] = to_f32<T>(raw[n + HIST - d].v[i]);
+        } else if (k.slot >= 0) {
+          sc_load<float, VEC>(h, rec + (size_t)(HIST + t - k.first - d) * p.C);
+        } else {
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) h[i] = 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) y[i] = fmaf(cw[j][i], h[i], y[i]);
+      }
     }
     if (k.slot >= 0 && p.rec.write) conv_leave<VEC>(p.rec, k, t, hist, p.C, c, now);
     if (c < p.out_w) sc_store<T, VEC>(reinterpret_cast<T*>(p.out) + (size_t)t * p.out_stride + c, y);
     if (p.slot_map != nullptr && c >= p.q_w) {
-      const long slot = p.slot_map[t];
+      const int slot = p.slot_map[t];
       if (slot < 0) continue;
       if (slot >= p.num_slots) {
         set_status(p.status, LL_ERR_SLOT_RANGE);
         continue;
       }
-      const long page = slot / p.page_size, place = slot - page * p.page_size;
+      const int page = slot / p.page_size, place = slot - page * p.page_size;
       const int kc = c - p.q_w;
       if (kc < p.k_w) {
         const int h = kc / p.hd;
@@ -484,13 +681,14 @@ __global__ void __launch_bounds__(32 * SC_TY) short_conv_kernel(const ShortConvP
 }
 
 template <typename T, int VEC, int TAPS>
-static int sc_launch(ShortConvParams p, int sms, cudaStream_t stream) {
+static int sc_launch(const ShortConvParams& p, int sms, cudaStream_t stream) {
   const int gx = (p.C + 32 * VEC - 1) / (32 * VEC);
-  // a token a thread while the step is short, up to four for long portions (a thread keeps its filters)
-  int per = (int)(((long)p.n * gx) / ((long)SC_TY * sms * 8));
-  p.per_thread = per < 1 ? 1 : per > 4 ? 4 : per;
-  const int rows = SC_TY * p.per_thread;
-  ll_launch(short_conv_kernel<T, VEC, TAPS>, dim3(gx, (p.n + rows - 1) / rows), dim3(32, SC_TY), 0, stream, p);
+  // a token a thread while the step is short, four (which keep their filters and share their rows) for long portions
+  if ((long)p.n * gx >= (long)SC_TY * sms * 8)
+    ll_launch(short_conv_kernel<T, VEC, TAPS, 4>, dim3(gx, (p.n + 4 * SC_TY - 1) / (4 * SC_TY)), dim3(32, SC_TY), 0,
+              stream, p);
+  else
+    ll_launch(short_conv_kernel<T, VEC, TAPS, 1>, dim3(gx, (p.n + SC_TY - 1) / SC_TY), dim3(32, SC_TY), 0, stream, p);
   return LL_LAUNCH_RESULT();
 }
 
@@ -510,7 +708,7 @@ static int sc_taps(const ShortConvParams& p, int sms, cudaStream_t stream) {
 extern "C" int ll_short_conv(int dtype, void* out, long out_stride, int out_w, const void* x, long x_stride, int C,
                              const float* w, int taps, int add, float* state, long state_stride, int write_state,
                              const int* token_req, const int* cu_q, const int* ctx_len, const int* req_slot,
-                             const int* slot_map, void* k_cache, void* v_cache, int q_w, int k_w, int hd, int vd, int nkv,
+                             int single, const int* slot_map, void* k_cache, void* v_cache, int q_w, int k_w, int hd, int vd, int nkv,
                              int page_size, long num_slots, int* status, int n, int sms, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (C <= 0 || taps < 1 || taps > 64 || state == nullptr || sms <= 0 || out_w < 0 || out_w > C ||
@@ -523,7 +721,7 @@ extern "C" int ll_short_conv(int dtype, void* out, long out_stride, int out_w, c
   p.w = w;
   p.taps = taps;
   p.C = C;
-  p.rec = {state, state_stride, write_state, token_req, cu_q, ctx_len, req_slot};
+  p.rec = {state, state_stride, write_state, token_req, cu_q, ctx_len, req_slot, single};
   p.out = out;
   p.out_stride = out_stride;
   p.out_w = out_w;
@@ -540,7 +738,6 @@ extern "C" int ll_short_conv(int dtype, void* out, long out_stride, int out_w, c
   p.num_slots = num_slots;
   p.status = status;
   p.n = n;
-  p.per_thread = 1;
   const int v = dtype == LL_DTYPE_BF16 ? 8 : 4;
   const bool wide = C % v == 0 && x_stride % v == 0 && out_stride % v == 0 && out_w % v == 0 && state_stride % 4 == 0 &&
                     (uintptr_t)x % 16 == 0 && (uintptr_t)out % 16 == 0 &&

@@ -1926,6 +1926,11 @@ def _conv_record(state: torch.Tensor, taps: int, channels: int) -> None:
           "a convolution's records are [request slots, conv_record_floats]")
 
 
+def _one_token_each(step, n: int) -> int:
+    """1 if every entry of the step brings one token, so that token t is entry t (the batch builder's arrays)."""
+    return 1 if step is not None and getattr(step, "num_single", -1) == n else 0
+
+
 def norm_conv(out: torch.Tensor, residual: torch.Tensor, weight: torch.Tensor, eps: float,
               res_out: Optional[torch.Tensor] = None, delta: Optional[torch.Tensor] = None,
               rows_in: Optional[torch.Tensor] = None, rows_w: Optional[torch.Tensor] = None,
@@ -1970,8 +1975,8 @@ def norm_conv(out: torch.Tensor, residual: torch.Tensor, weight: torch.Tensor, e
         "ll_norm_conv", c_int(_dtype_code(out)), _ptr(out), _ptr(res_out), _ptr(residual), _ptr(delta), _ptr(partial),
         c_int(parts), c_long(part_stride), _ptr(rows_in), _ptr(rows_w if rows_in is not None else None), _ptr(extra),
         _ptr(weight), c_float(eps), _ptr(conv_w), c_int(taps), _ptr(state if conv_w is not None else None), c_long(stride),
-        c_int(1 if write_state else 0), _ptr(token_req), _ptr(cu_q), _ptr(ctx_len), _ptr(req_slot), _ptr(rows), c_int(n),
-        c_int(W), c_int(sm_count(out.device)), _stream())
+        c_int(1 if write_state else 0), _ptr(token_req), _ptr(cu_q), _ptr(ctx_len), _ptr(req_slot),
+        c_int(_one_token_each(step, n)), _ptr(rows), c_int(n), c_int(W), c_int(sm_count(out.device)), _stream())
 
 
 def short_conv(out: Optional[torch.Tensor], x: torch.Tensor, conv_w: torch.Tensor, state: torch.Tensor, step,
@@ -2008,7 +2013,7 @@ def short_conv(out: Optional[torch.Tensor], x: torch.Tensor, conv_w: torch.Tenso
         "ll_short_conv", c_int(_dtype_code(x)), _ptr(out), c_long(out_stride), c_int(out_w), _ptr(x), c_long(x.stride(0)),
         c_int(C), _ptr(conv_w), c_int(taps), c_int(1 if add_input else 0), _ptr(state), c_long(state.stride(0)),
         c_int(1 if write_state else 0), _ptr(step.token_req), _ptr(step.cu_q), _ptr(step.ctx_len), _ptr(step.req_slot),
-        _ptr(slot_map), _ptr(k_cache), _ptr(v_cache), c_int(q_w), c_int(k_w), c_int(hd), c_int(vd), c_int(nkv),
+        c_int(_one_token_each(step, n)), _ptr(slot_map), _ptr(k_cache), _ptr(v_cache), c_int(q_w), c_int(k_w), c_int(hd), c_int(vd), c_int(nkv),
         c_int(page_size), c_long(num_slots), _ptr(status), c_int(n), c_int(sm_count(x.device)), _stream())
 
 
