@@ -47,12 +47,14 @@ class RunStep:
     mixer works on: ``None`` gives the entry a plane of its own; the index of
     an earlier entry makes it read that entry's plane without writing to it.
     ``add_embedding``: the embedding's output is added to the residual before
-    the layer runs (a range of layers that runs again starts with it).
+    the layer runs (a range of layers that runs again starts with it);
+    ``add_row``: that row of ``ModelSpec.pass_rows`` is, for every token.
     """
 
     layer: int
     cache: Optional[int] = None
     add_embedding: bool = False
+    add_row: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -69,3 +71,4 @@ class ModelSpec:
     final_norm: PartSpec
     head: PartSpec
     eos_token_ids: Tuple[int, ...] = ()
+    pass_rows: Optional[PartSpec] = None

@@ -96,7 +96,7 @@ __global__ void act_mul_kernel(T* __restrict__ out, const T* __restrict__ gu, lo
 extern "C" int ll_act_mul(int dtype, void* out, const void* gate_up, int num_tokens, int inter, int act,
                           float limit, float alpha, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
-  if (act < 0 || act > 2) return (int)cudaErrorInvalidValue;
+  if (act < 0 || act > 3) return (int)cudaErrorInvalidValue;
   const long total = (long)num_tokens * inter;
   const int blocks = (int)min((total + 255) / 256, (long)silu_device_sms() * 16);
   LL_DISPATCH_DTYPE(dtype, ll_launch(act_mul_kernel<T>, dim3(blocks), dim3(256), 0, stream, (T*)out,

@@ -17,6 +17,10 @@
 //   o_h       = sum_j w_h[j] v_(h / group)[j]  (* sigmoid(gate[h]) with a gate a head, or every channel of the
 //               head times the sigmoid of its own gate input)
 //
+// Pairs (`pairs`): the query heads come in neighbouring pairs, two score maps over the same keys and values, and the
+// heads' outputs are combined: z = o_even - lambda o_odd, then z / sqrt(mean(z^2) + eps) * post over the head's vd
+// values, then the gate; nh / 2 heads come out, and a gate is a number a head of those.
+//
 // One block a token.  Without `mix` a block works on one kv head and its query heads; with it, on all heads
 // at once, since every head's score needs every other head's.  Keys are walked in tiles that start at
 // multiples of the tile size, so the order of every sum depends on the position only: the result for a
@@ -38,7 +42,8 @@ attention_modulated_kernel(T* __restrict__ out, long out_stride, const T* __rest
                            const float* __restrict__ temp, const float* __restrict__ mix, int tk, int* status,
                            const float* __restrict__ sink_val, const float* __restrict__ rel, int nd, int keep,
                            float cap, float qt_coef, int qt_every, long gate_stride, int gate_channels,
-                           float out_scale, const float* __restrict__ slope) {
+                           float out_scale, const float* __restrict__ slope, int pairs, float lambda, float post,
+                           float pair_eps) {
   extern __shared__ float smem[];
   LL_PDL_WAIT();
   LL_PDL_TRIGGER();
@@ -59,14 +64,15 @@ attention_modulated_kernel(T* __restrict__ out, long out_stride, const T* __rest
   float* m_s = ps + hb * 32;                      // [hb]
   float* l_s = m_s + hb;                          // [hb]
   float* alpha_s = l_s + hb;                      // [hb]
-  float* mix_s = alpha_s + hb;                    // [hb][hb] with mix
+  float* mix_s = alpha_s + hb;                    // [hb][hb] with mix; [hb][vd] with pairs: the outputs
 
   const int entry = token_req[t];
   const int slot = entry >= 0 ? req_slot[entry] : -1;
   const int p = positions[t];
-  T* o_row = out + (size_t)t * out_stride + (size_t)head0 * vd;
+  const int fold = pairs ? 2 : 1;                 // query heads an output head
+  T* o_row = out + (size_t)t * out_stride + (size_t)(head0 / fold) * vd;
   if (slot < 0 || p < 0) {  // padding entry of a captured batch: defined output, no reads
-    for (int i = tid; i < hb * vd; i += AM_THREADS) o_row[i] = from_f32<T>(0.f);
+    for (int i = tid; i < hb / fold * vd; i += AM_THREADS) o_row[i] = from_f32<T>(0.f);
     return;
   }
   const int* bt = block_table + (size_t)slot * bt_stride;
@@ -172,7 +178,28 @@ attention_modulated_kernel(T* __restrict__ out, long out_stride, const T* __rest
   }
   __syncthreads();
   // ---- normalise, gate and write ----
-  const T* g_row = gate ? gate + (size_t)t * gate_stride + (gate_channels ? (size_t)head0 * vd : (size_t)head0) : nullptr;
+  const T* g_row = gate ? gate + (size_t)t * gate_stride + (gate_channels ? (size_t)head0 * vd : (size_t)(head0 / fold)) : nullptr;
+  if (pairs) {
+    float* fin = mix_s;
+#pragma unroll
+    for (int c = 0; c < ACC; ++c) {
+      const int idx = tid + c * AM_THREADS;
+      if (idx < outs) fin[idx] = acc[c] / l_s[idx / vd];
+    }
+    __syncthreads();
+    for (int h = warp; h < hb / 2; h += AM_WARPS) {       // a warp an output head
+      float* z = fin + (size_t)(2 * h) * vd;
+      float ss = 0.f;
+      for (int d = lane; d < vd; d += 32) {
+        z[d] -= lambda * z[vd + d];
+        ss += z[d] * z[d];
+      }
+      float f = post / sqrtf(warp_sum(ss) / (float)vd + pair_eps) * out_scale;
+      if (g_row) f *= 1.0f / (1.0f + expf(-to_f32<T>(g_row[h])));
+      for (int d = lane; d < vd; d += 32) o_row[(size_t)h * vd + d] = from_f32<T>(z[d] * f);
+    }
+    return;
+  }
 #pragma unroll
   for (int c = 0; c < ACC; ++c) {
     const int idx = tid + c * AM_THREADS;
@@ -187,10 +214,10 @@ attention_modulated_kernel(T* __restrict__ out, long out_stride, const T* __rest
 
 // Keys a tile for these sizes: the largest of 32, 16, 8 whose tile fits in shared memory.  It depends on the
 // sizes only, never on the step, so a position's sums keep their order.
-static int am_tile_keys(int hb, int nkb, int hd, int vd, size_t* smem_out) {
+static int am_tile_keys(int hb, int nkb, int hd, int vd, int pairs, size_t* smem_out) {
   for (int tk = 32; tk >= 8; tk >>= 1) {
     const size_t floats = (size_t)hb * hd + (size_t)tk * nkb * (hd + 1 + vd) + (size_t)hb * 64 + 3 * (size_t)hb +
-                          (size_t)hb * hb;
+                          (pairs ? (size_t)hb * vd : (size_t)hb * hb);
     if (floats * sizeof(float) <= 200 * 1024) {
       *smem_out = floats * sizeof(float);
       return tk;
@@ -219,15 +246,16 @@ extern "C" int ll_attention_modulated(int dtype, void* out, long out_stride, con
                                       const float* temp, const float* mix, int* status, const float* sink_val,
                                       const float* rel, int nd, int keep, float cap, float qt_coef, int qt_every,
                                       long gate_stride, int gate_channels, float out_scale, const float* slope,
-                                      cudaStream_t stream) {
+                                      int pairs, float lambda, float post, float pair_eps, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (hd <= 0 || vd <= 0 || nkv <= 0 || nh % nkv != 0 || page_size <= 0 || mask < 0 || mask > 2 ||
-      (rel != nullptr && nd <= 0) || keep < 0)
+      (rel != nullptr && nd <= 0) || keep < 0 ||
+      (pairs && (mix != nullptr || gate_channels || (nh / nkv) % 2 != 0)))
     return (int)cudaErrorInvalidValue;
   const int group = nh / nkv;
   const int hb = mix ? nh : group, nkb = mix ? nkv : 1;
   size_t smem = 0;
-  const int tk = am_tile_keys(hb, nkb, hd, vd, &smem);
+  const int tk = am_tile_keys(hb, nkb, hd, vd, pairs, &smem);
   const int per_thread = (hb * vd + AM_THREADS - 1) / AM_THREADS;
   if (tk == 0 || per_thread > 32) return (int)cudaErrorInvalidValue;
   dim3 grid(num_tokens, mix ? 1 : nkv);
@@ -240,7 +268,7 @@ extern "C" int ll_attention_modulated(int dtype, void* out, long out_stride, con
               (const T*)q, q_stride, (const T*)gate, (const T*)k_cache, (const T*)v_cache, block_table, bt_stride,  \
               token_req, req_slot, positions, nh, nkv, hd, vd, page_size, num_pages, mask, mask_size, sink, scale,  \
               temp, mix, tk, status, sink_val, rel, nd, keep, cap, qt_coef, qt_every, gate_stride, gate_channels,   \
-              out_scale, slope);                                                                                    \
+              out_scale, slope, pairs, lambda, post, pair_eps);                                                                                    \
   } while (0)
   LL_DISPATCH_DTYPE(dtype, {
     if (per_thread <= 4) AM_LAUNCH(4);

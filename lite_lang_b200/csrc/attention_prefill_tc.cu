@@ -33,6 +33,10 @@
 // window), the softmax warps overwrite those keys' rows of V in shared memory with zeros before the
 // product is issued.  A table entry of a key that a row does see must name a page of the pool; one that
 // does not sets LL_ERR_PAGE_RANGE.
+//
+// Pairs: neighbouring query heads (2a, 2a + 1) are two score maps over the same keys and values and come out as one head,
+// z = o_even - lambda o_odd, z / sqrt(mean(z^2) + eps) * post (float32, before the gate and the one rounding).  Their rows
+// are neighbouring lanes of a warp.
 #include "tc05.cuh"
 
 #define AT_THREADS 192
@@ -58,6 +62,8 @@ struct AttnTcParams {
   // a gate a head on the output (optional): out[token, head] *= sigmoid(gate[token * gate_stride + head]), float32
   const bf16* gate;
   long gate_stride;
+  int pairs;           // heads 2a and 2a + 1 come out as one (half as many heads in out and gate)
+  float lambda, post, pair_eps;
   float* scratch;      // [row blocks * nkv * nsplit][HD + 2][128]
   int* counters;       // [row blocks * nkv], zero between launches
   int* status;
@@ -363,7 +369,7 @@ attn_prefill_tc_kernel(const AttnTcParams p, const __grid_constant__ CUtensorMap
     AT_FENCE_AFTER();
     // ---- the splits of a row block meet in scratch memory; the last one to arrive goes on ----
     bool finish = true;
-    float inv;
+    float inv, post = 1.0f;
     const size_t part0 = ((size_t)rb_step * p.nkv + kvh) * p.nsplit;     // this row block's first partial
     constexpr int PSTRIDE = (HD + 2) * 128;   // floats a partial: column-major [HD + 2][128 rows] (O, maximum, sum),
                                               // so that a warp's 32 rows read and write 128 contiguous bytes
@@ -428,7 +434,25 @@ attn_prefill_tc_kernel(const AttnTcParams p, const __grid_constant__ CUtensorMap
     } else {
       inv = l_run > 0.f ? 1.0f / l_run : 0.f;
     }
-    if (finish && p.gate != nullptr) {
+    if (finish && p.pairs) {
+      float ss = 0.f;
+#pragma unroll
+      for (int c0 = 0; c0 < HD; c0 += 32) {
+        float v[32];
+        at_ld32(tmem_o + lane_addr + c0, v);
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          const float own = v[i] * inv;
+          const float z = own - p.lambda * __shfl_xor_sync(0xffffffffu, own, 1);
+          ss = fmaf(z, z, ss);
+        }
+      }
+      post = p.post / sqrtf(ss / (float)HD + p.pair_eps);
+      if (p.gate != nullptr && row_ok) {
+        const float gv = __bfloat162float(p.gate[(size_t)(tok0 + t) * p.gate_stride + (size_t)((kvh * p.group + g) >> 1)]);
+        post *= 1.0f / (1.0f + expf(-gv));
+      }
+    } else if (finish && p.gate != nullptr) {
       const int tt = r / p.group, gg = r - tt * p.group;
       if (r < p.tpb * p.group && tt < ntok) {
         const float gv = __bfloat162float(p.gate[(size_t)(tok0 + tt) * p.gate_stride + (size_t)(kvh * p.group + gg)]);
@@ -443,12 +467,18 @@ attn_prefill_tc_kernel(const AttnTcParams p, const __grid_constant__ CUtensorMap
         float v[32];
         at_ld32(tmem_o + lane_addr + c0, v);
 #pragma unroll
+        for (int i = 0; i < 32; ++i) v[i] *= inv;
+        if (p.pairs) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) v[i] = (v[i] - p.lambda * __shfl_xor_sync(0xffffffffu, v[i], 1)) * post;
+        }
+#pragma unroll
         for (int cc = 0; cc < 4; ++cc) {
           const int c = c0 / 8 + cc;
           unsigned w[4];
 #pragma unroll
           for (int i = 0; i < 4; ++i) {
-            const __nv_bfloat162 h = __floats2bfloat162_rn(v[8 * cc + 2 * i] * inv, v[8 * cc + 2 * i + 1] * inv);
+            const __nv_bfloat162 h = __floats2bfloat162_rn(v[8 * cc + 2 * i], v[8 * cc + 2 * i + 1]);
             w[i] = *reinterpret_cast<const unsigned*>(&h);
           }
           *reinterpret_cast<uint4*>(orow + (((c & ~7) | ((c ^ r) & 7)) << 4)) = make_uint4(w[0], w[1], w[2], w[3]);
@@ -461,9 +491,10 @@ attn_prefill_tc_kernel(const AttnTcParams p, const __grid_constant__ CUtensorMap
     for (int idx = e; finish && idx < 128 * CPR; idx += 128) {
       const int rr = idx / CPR, c = idx % CPR;
       const int tt = rr / p.group, gg = rr - tt * p.group;
-      if (rr < p.tpb * p.group && tt < ntok) {
+      if (rr < p.tpb * p.group && tt < ntok && !(p.pairs && (rr & 1))) {
         const uint4 v = *reinterpret_cast<const uint4*>(q_s + rr * (HD * 2) + (((c & ~7) | ((c ^ rr) & 7)) << 4));
-        *reinterpret_cast<uint4*>(p.out + (size_t)(tok0 + tt) * p.out_stride + (size_t)(kvh * p.group + gg) * HD + 8 * c) = v;
+        const int head = kvh * p.group + gg;
+        *reinterpret_cast<uint4*>(p.out + (size_t)(tok0 + tt) * p.out_stride + (size_t)(p.pairs ? head >> 1 : head) * HD + 8 * c) = v;
       }
     }
     (void)g;
@@ -502,9 +533,10 @@ static int at_run(void* out, long out_stride, const void* q, long q_stride, int 
                   const void* v_cache, const int* block_table, int bt_stride, const int* cu_q, const int* ctx_len,
                   const int* req_slot, int n_entries, int row_blocks, int nh, int nkv, int hd, int page_size,
                   int num_pages, int window, float scale, int nsplit, int split_len, float* scratch, int* counters,
-                  const void* gate, long gate_stride, int* status, cudaStream_t stream) {
+                  const void* gate, long gate_stride, int pairs, float lambda, float post, float pair_eps, int* status,
+                  cudaStream_t stream) {
   if (row_blocks <= 0 || n_entries <= 0) return 0;
-  if ((hd != 64 && hd != 128) || nkv <= 0 || nh % nkv != 0 || nkv > 65535 || nh / nkv > 128)
+  if ((hd != 64 && hd != 128) || nkv <= 0 || nh % nkv != 0 || nkv > 65535 || nh / nkv > 128 || (pairs && (nh / nkv) % 2 != 0))
     return (int)cudaErrorInvalidValue;
   if (!(page_size == 8 || page_size == 16 || page_size == 32 || (page_size > 0 && page_size % 64 == 0)))
     return (int)cudaErrorInvalidValue;
@@ -536,6 +568,10 @@ static int at_run(void* out, long out_stride, const void* q, long q_stride, int 
   p.counters = counters;
   p.gate = (const bf16*)gate;
   p.gate_stride = gate_stride;
+  p.pairs = pairs;
+  p.lambda = lambda;
+  p.post = post;
+  p.pair_eps = pair_eps;
   p.status = status;
 
   CUtensorMap qmap, kmap, vmap;
@@ -580,7 +616,7 @@ extern "C" int ll_attn_prefill_tc(void* out, long out_stride, const void* q, lon
                                   int* status, cudaStream_t stream) {
   return at_run(out, out_stride, q, q_stride, num_tokens, k_cache, v_cache, block_table, bt_stride, cu_q, ctx_len, req_slot,
                 n_entries, row_blocks, nh, nkv, hd, page_size, num_pages, window, scale, nsplit, split_len, scratch,
-                counters, nullptr, 0, status, stream);
+                counters, nullptr, 0, 0, 0.f, 0.f, 0.f, status, stream);
 }
 
 // The same with a gate a head on the output: gate is bfloat16, gate[token * gate_stride + head], and every head's
@@ -594,5 +630,19 @@ extern "C" int ll_attn_prefill_tc_gated(void* out, long out_stride, const void* 
                                         cudaStream_t stream) {
   return at_run(out, out_stride, q, q_stride, num_tokens, k_cache, v_cache, block_table, bt_stride, cu_q, ctx_len, req_slot,
                 n_entries, row_blocks, nh, nkv, hd, page_size, num_pages, window, scale, nsplit, split_len, scratch,
-                counters, gate, gate_stride, status, stream);
+                counters, gate, gate_stride, 0, 0.f, 0.f, 0.f, status, stream);
+}
+
+// The same for heads in pairs (see the head of this file): out is [tokens, nh / 2 * hd], gate (or null) a number for each of
+// those heads.
+extern "C" int ll_attn_prefill_tc_pairs(void* out, long out_stride, const void* q, long q_stride, int num_tokens,
+                                        const void* k_cache, const void* v_cache, const int* block_table, int bt_stride,
+                                        const int* cu_q, const int* ctx_len, const int* req_slot, int n_entries,
+                                        int row_blocks, int nh, int nkv, int hd, int page_size, int num_pages,
+                                        int window, float scale, int nsplit, int split_len, float* scratch,
+                                        int* counters, const void* gate, long gate_stride, float lambda, float post,
+                                        float pair_eps, int* status, cudaStream_t stream) {
+  return at_run(out, out_stride, q, q_stride, num_tokens, k_cache, v_cache, block_table, bt_stride, cu_q, ctx_len, req_slot,
+                n_entries, row_blocks, nh, nkv, hd, page_size, num_pages, window, scale, nsplit, split_len, scratch,
+                counters, gate, gate_stride, 1, lambda, post, pair_eps, status, stream);
 }

@@ -30,6 +30,10 @@
 // stages that hold them are walked before the window's: by part 0 where the keys are split); a sink of a learned
 // score a head in the place of 0; a sigmoid gate a channel in the place of one a head; a constant on the output; a
 // penalty that grows with the distance by a slope a head, taken off after the cap.
+//
+// Pairs: neighbouring query heads (2a, 2a + 1) are two score maps over the same keys and values and come out as one head,
+// z = o_even - lambda o_odd, z / sqrt(mean(z^2) + eps) * post (before the gate).  The two rows of a pair are neighbours
+// among a warp's rows, so the lanes that hold them exchange (or, with splits, the join's block makes both).
 #include "common.cuh"
 
 #define AS_WARPS 8
@@ -70,6 +74,8 @@ struct AttnShapedParams {
   int gate_channels;      // the gate is a number a channel: token t, head h, channel d at gate[t * gate_stride + h * VD + d]
   float out_scale;
   const float* slope;     // optional [nh]: a key n positions back has slope * n taken off its score (natural units)
+  int pairs;              // heads 2a and 2a + 1 come out as one (nh / 2 heads in out and gate)
+  float lambda, post, pair_eps;
 };
 #define AS_LOG2E 1.4426950408889634f
 // tanh from exp2 and a division: absolute error of a few 1e-7
@@ -163,8 +169,8 @@ __global__ void __launch_bounds__(AS_THREADS) attn_shaped_kernel(const AttnShape
     if (!split) {
 #pragma unroll
       for (int i = 0; i < 2; ++i)
-        if (validr[i]) {
-          bf16* o = p.out + (size_t)(tok0 + tokr[i]) * p.out_stride + (size_t)headr[i] * VD;
+        if (validr[i] && !(p.pairs && (headr[i] & 1))) {
+          bf16* o = p.out + (size_t)(tok0 + tokr[i]) * p.out_stride + (size_t)(p.pairs ? headr[i] >> 1 : headr[i]) * VD;
           for (int d = c; d < VD; d += 4) o[d] = __float2bfloat16_rn(0.f);
         }
     }
@@ -465,9 +471,33 @@ __global__ void __launch_bounds__(AS_THREADS) attn_shaped_kernel(const AttnShape
   for (int i = 0; i < 2; ++i) {
     const float l = l_run[i] + (sink_here ? as_exp2(sink_log2[i] - m_run[i]) : 0.f);
     inv[i] = (l > 0.f ? 1.0f / l : 0.f) * p.out_scale;
-    if (p.gate && !p.gate_channels) {
+    if (p.gate && !p.gate_channels && !p.pairs) {
       const float gv = __bfloat162float(p.gate[(size_t)(tok0 + tokr[i]) * p.gate_stride + headr[i]]);
       inv[i] *= 1.0f / (1.0f + expf(-gv));
+    }
+  }
+  if (p.pairs) {
+    // rows g and g ^ 1 are a pair: the even one takes the odd one's values from the lane four away (all lanes of the
+    // warp go through this; rows that do not exist are not written)
+    float ss[2] = {0.f, 0.f};
+#pragma unroll
+    for (int Tn = 0; Tn < NT; ++Tn)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) {
+        const float own = o_acc[Tn][x] * inv[x >> 1];
+        const float other = __shfl_xor_sync(0xffffffffu, own, 4);
+        o_acc[Tn][x] = own - p.lambda * other;
+        ss[x >> 1] = fmaf(o_acc[Tn][x], o_acc[Tn][x], ss[x >> 1]);
+      }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], 1);
+      ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], 2);
+      inv[i] = p.post / sqrtf(ss[i] / (float)VD + p.pair_eps);
+      if (p.gate) {
+        const float gv = __bfloat162float(p.gate[(size_t)(tok0 + tokr[i]) * p.gate_stride + (headr[i] >> 1)]);
+        inv[i] *= 1.0f / (1.0f + expf(-gv));
+      }
     }
   }
   // each warp has 16 rows x VD bfloat16 of staging space (the buffers are free now: all warps passed the last
@@ -497,7 +527,11 @@ __global__ void __launch_bounds__(AS_THREADS) attn_shaped_kernel(const AttnShape
     const int r = rw0 + row;
     if (r < total_rows) {
       const int tok = r / p.group;
-      const int head = kvh * p.group + (r - tok * p.group);
+      int head = kvh * p.group + (r - tok * p.group);
+      if (p.pairs) {
+        if (head & 1) continue;
+        head >>= 1;
+      }
       const uint4 v = *reinterpret_cast<const uint4*>(stage + row * (VD + 8) + 8 * chunk);
       *reinterpret_cast<uint4*>(p.out + (size_t)(tok0 + tok) * p.out_stride + (size_t)head * VD + 8 * chunk) = v;
     }
@@ -508,19 +542,7 @@ __global__ void __launch_bounds__(AS_THREADS) attn_shaped_kernel(const AttnShape
 // M the largest maximum (0 at least with a sink), times the head's gate.  How many parts a row has follows
 // from its position as in the first kernel.  One block a (entry, head), a thread a value channel.
 template <int VD>
-__global__ void __launch_bounds__(VD) attn_shaped_join_kernel(const AttnShapedParams p) {
-  LL_PDL_WAIT();
-  LL_PDL_TRIGGER();
-  const int e = blockIdx.x, head = blockIdx.y, d = threadIdx.x;
-  const int tok = p.cu_q[e];
-  bf16* o = p.out + (size_t)tok * p.out_stride + (size_t)head * VD;
-  if (p.req_slot[e] < 0) {
-    o[d] = __float2bfloat16_rn(0.f);
-    return;
-  }
-  const int pos = p.ctx_len[e];
-  const int stages = pos / AS_TK - as_first_visible(p.mask, p.mask_size, pos) / AS_TK + 1;
-  const int parts = min(p.nsplit, (stages + p.span - 1) / p.span);
+__device__ __forceinline__ float as_join_row(const AttnShapedParams& p, int tok, int head, int parts, int d) {
   const float* src = p.part + ((size_t)tok * p.nh + head) * p.nsplit * (VD + 2);
   const float sink_log2 = p.sink_val ? p.sink_val[head] * AS_LOG2E : 0.f;
   float M = p.sink ? sink_log2 : -INFINITY;
@@ -533,7 +555,31 @@ __global__ void __launch_bounds__(VD) attn_shaped_join_kernel(const AttnShapedPa
     L = fmaf(s[VD + 1], w, L);
     acc = fmaf(s[d], w, acc);
   }
-  float r = (L > 0.f ? acc / L : 0.f) * p.out_scale;
+  return (L > 0.f ? acc / L : 0.f) * p.out_scale;
+}
+
+template <int VD>
+__global__ void __launch_bounds__(VD) attn_shaped_join_kernel(const AttnShapedParams p) {
+  __shared__ float scratch[32];
+  LL_PDL_WAIT();
+  LL_PDL_TRIGGER();
+  const int e = blockIdx.x, head = blockIdx.y, d = threadIdx.x;      // (head: of the output)
+  const int tok = p.cu_q[e];
+  bf16* o = p.out + (size_t)tok * p.out_stride + (size_t)head * VD;
+  if (p.req_slot[e] < 0) {
+    o[d] = __float2bfloat16_rn(0.f);
+    return;
+  }
+  const int pos = p.ctx_len[e];
+  const int stages = pos / AS_TK - as_first_visible(p.mask, p.mask_size, pos) / AS_TK + 1;
+  const int parts = min(p.nsplit, (stages + p.span - 1) / p.span);
+  float r;
+  if (p.pairs) {
+    r = as_join_row<VD>(p, tok, 2 * head, parts, d) - p.lambda * as_join_row<VD>(p, tok, 2 * head + 1, parts, d);
+    r *= p.post / sqrtf(block_sum(r * r, scratch) / (float)VD + p.pair_eps);
+  } else {
+    r = as_join_row<VD>(p, tok, head, parts, d);
+  }
   if (p.gate)
     r *= 1.0f / (1.0f + expf(-__bfloat162float(p.gate[(size_t)tok * p.gate_stride +
                                                        (p.gate_channels ? (size_t)head * VD + d : (size_t)head)])));
@@ -553,7 +599,8 @@ extern "C" long ll_attn_shaped_smem(int nkv, int hd, int vd, int mixed) {
 // out [tokens, nh * vd].  k_cache [pages, nkv, page_size, hd], v_cache [pages, nkv, page_size, vd].
 // cu_q, ctx_len, req_slot: the entries; row_blocks = sum over them of ceil(q_len * group / 128).
 // sink_val (optional float32 [nh]), rel (optional float32 [nd, nh]), keep, cap (0: none), qt_coef / qt_every
-// (0: none), gate_channels, out_scale, slope (optional float32 [nh]): see the head of this file.
+// (0: none), gate_channels, out_scale, slope (optional float32 [nh]), pairs with lambda, post and pair_eps: see the head of
+// this file.
 // mask 0 causal, 1 window, 2 chunks of mask_size.  nsplit > 1 (every entry brings one token): the keys of a
 // row are cut into parts of `span` stages of 64 keys; part float32 [tokens, nh, nsplit, vd + 2].
 extern "C" int ll_attn_shaped(void* out, long out_stride, const void* q, long q_stride, int mixed, const void* gate,
@@ -563,14 +610,16 @@ extern "C" int ll_attn_shaped(void* out, long out_stride, const void* q, long q_
                               int page_size, int num_pages, int mask, int mask_size, int sink, float scale, int nsplit,
                               int span, float* part, int* status, const float* sink_val, const float* rel, int nd,
                               int keep, float cap, float qt_coef, int qt_every, int gate_channels, float out_scale,
-                              const float* slope, cudaStream_t stream) {
+                              const float* slope, int pairs, float lambda, float post, float pair_eps,
+                              cudaStream_t stream) {
   if (row_blocks <= 0 || n_entries <= 0) return 0;
   const long smem = ll_attn_shaped_smem(nkv, hd, vd, mixed);
   if (smem == 0 || page_size % 16 != 0 || nh % nkv != 0 || nkv > 65535 || mask < 0 || mask > 2 ||
       (mask != 0 && mask_size <= 0) || nsplit < 1 || nsplit > 65535 || (nsplit > 1 && (part == nullptr || span < 1)))
     return (int)cudaErrorInvalidValue;
   if ((q_stride % 8) != 0 || (out_stride % 8) != 0 || (rel != nullptr && nd <= 0) || keep < 0 ||
-      (mixed && (rel != nullptr || cap > 0.f || sink_val != nullptr || slope != nullptr)))
+      (mixed && (rel != nullptr || cap > 0.f || sink_val != nullptr || slope != nullptr)) ||
+      (pairs && (mixed || gate_channels || (nh / nkv) % 2 != 0)))
     return (int)cudaErrorInvalidValue;
   AttnShapedParams p;
   p.q = (const bf16*)q;
@@ -612,6 +661,10 @@ extern "C" int ll_attn_shaped(void* out, long out_stride, const void* q, long q_
   p.gate_channels = gate_channels;
   p.out_scale = out_scale;
   p.slope = slope;
+  p.pairs = pairs;
+  p.lambda = lambda;
+  p.post = post;
+  p.pair_eps = pair_eps;
   dim3 grid(row_blocks, nkv, nsplit);
 #define AS_LAUNCH(HD_, VD_, MIX_)                                                                                  \
   do {                                                                                                             \
@@ -633,7 +686,7 @@ extern "C" int ll_attn_shaped(void* out, long out_stride, const void* q, long q_
   int rc = LL_LAUNCH_RESULT();
   if (rc != 0 || nsplit == 1) return rc;
   // the rows of the single tokens: row_blocks counts ceil(group / 128) blocks an entry here
-  dim3 jgrid(n_entries, nh);
+  dim3 jgrid(n_entries, pairs ? nh / 2 : nh);
   if (vd == 64) ll_launch(attn_shaped_join_kernel<64>, jgrid, dim3(64), 0, stream, p);
   else ll_launch(attn_shaped_join_kernel<128>, jgrid, dim3(128), 0, stream, p);
   return LL_LAUNCH_RESULT();

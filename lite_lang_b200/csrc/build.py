@@ -52,6 +52,7 @@ LIBRARIES: Dict[str, Tuple[Tuple[str, ...], Tuple[str, ...]]] = {
     "attn_mod": (("qkv_norm_rotate_store.cu", "attention_modulated.cu"), ()),
     "attn_shaped": (("attention_shaped_mma.cu",), ()),
     "short_conv": (("short_conv.cu",), ()),
+    "sandwich": (("sandwich_norm.cu",), ()),
 }
 
 _INCLUDE = re.compile(r'^\s*#\s*include\s+"([^"]+)"', re.M)

@@ -75,7 +75,7 @@ __device__ __forceinline__ void set_status(int* status, int code) {
 }
 
 // The activation of a gated product: 0 silu(g) u, 1 relu(g) u, 2 (clamped swish) a sigmoid(alpha a) (c + 1) with
-// a = min(g, limit), c = clamp(u, -limit, limit).
+// a = min(g, limit), c = clamp(u, -limit, limit), 3 gelu(g) u (gelu in its tanh form).
 struct GateAct {
   int act;
   float limit, alpha;
@@ -85,7 +85,12 @@ __device__ __forceinline__ float ll_clamped_swish(float g, float u, float limit,
   const float c = fminf(fmaxf(u, -limit), limit);
   return a / (1.0f + expf(-alpha * a)) * (c + 1.0f);
 }
+// gelu in its tanh form, 0.5 z (1 + tanh(y)) = z / (1 + e^(-2y)) with y = sqrt(2/pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float ll_gelu_tanh(float z) {
+  return z / (1.0f + expf(-1.5957691216057308f * (z + 0.044715f * z * z * z)));
+}
 __device__ __forceinline__ float ll_gated(float g, float u, const GateAct& k) {
+  if (k.act == 3) return ll_gelu_tanh(g) * u;
   if (k.act == 2) return ll_clamped_swish(g, u, k.limit, k.alpha);
   return (k.act == 1 ? fmaxf(g, 0.f) : g / (1.0f + expf(-g))) * u;
 }
@@ -96,6 +101,7 @@ __device__ __forceinline__ float ll_gated_fast(float g, float u, const GateAct& 
     const float c = fminf(fmaxf(u, -k.limit), k.limit);
     return __fdividef(a, 1.0f + __expf(-k.alpha * a)) * (c + 1.0f);
   }
+  if (k.act == 3) return __fdividef(g, 1.0f + __expf(-1.5957691216057308f * (g + 0.044715f * g * g * g))) * u;
   return k.act == 1 ? fmaxf(g, 0.f) * u : __fdividef(g, 1.0f + __expf(-g)) * u;
 }
 

@@ -659,8 +659,8 @@ extern "C" int ll_gemm_pair(void* out, long out_stride, const void* x, long x_st
   p.N = N;
   p.K = K;
   p.status = status;
-  if (gated < 0 || gated > 3) return (int)cudaErrorInvalidValue;
-  p.gate = {gated > 0 ? gated - 1 : 0, limit, alpha};      // (gated: 1 SiLU, 2 ReLU, 3 clamped swish)
+  if (gated < 0 || gated > 4) return (int)cudaErrorInvalidValue;
+  p.gate = {gated > 0 ? gated - 1 : 0, limit, alpha};      // (gated: 1 SiLU, 2 ReLU, 3 clamped swish, 4 gelu)
   p.act = 0;
   p.vec_ok = ((uintptr_t)out % 16 == 0 && out_stride % 8 == 0 && N % 8 == 0) ? 1 : 0;
   p.bias = nullptr;

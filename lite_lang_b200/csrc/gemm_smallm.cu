@@ -182,8 +182,8 @@ extern "C" int ll_gemm_smallm(void* out, long out_stride, int out_f32, const voi
                               int M, int N, int K, int gated, float limit, float alpha, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return 0;
   if (M > 64 || K <= 0 || (K % 32) != 0 || (x_stride % 8) != 0) return (int)cudaErrorInvalidValue;
-  if (gated < 0 || gated > 3) return (int)cudaErrorInvalidValue;
-  const GateAct act = {gated > 0 ? gated - 1 : 0, limit, alpha};      // (gated: 1 SiLU, 2 ReLU, 3 clamped swish)
+  if (gated < 0 || gated > 4) return (int)cudaErrorInvalidValue;
+  const GateAct act = {gated > 0 ? gated - 1 : 0, limit, alpha};      // (gated: 1 SiLU, 2 ReLU, 3 clamped swish, 4 gelu)
   if (gated) {
     if (out_f32) return (int)cudaErrorInvalidValue;
     return gs_dispatch_m<true, bf16>(out, out_stride, x, x_stride, w, M, N, K, act, stream);

@@ -693,7 +693,7 @@ extern "C" int ll_gemm_stream(void* out, long out_stride, int out_f32, const voi
   p.M = M;
   p.N = N;
   p.K = K;
-  if (act > 2) return (int)cudaErrorInvalidValue;
+  if (act > 3) return (int)cudaErrorInvalidValue;
   p.gate = {act, limit, alpha};
   p.row_act = row_act;
   p.status = status;

@@ -442,8 +442,8 @@ extern "C" int ll_gemm_tc(void* out, long out_stride, int out_f32, const void* x
   p.N = N;
   p.K = K;
   p.status = status;
-  if (gated < 0 || gated > 3) return (int)cudaErrorInvalidValue;
-  p.gate = {gated > 0 ? gated - 1 : 0, limit, alpha};      // (gated: 1 SiLU, 2 ReLU, 3 clamped swish)
+  if (gated < 0 || gated > 4) return (int)cudaErrorInvalidValue;
+  p.gate = {gated > 0 ? gated - 1 : 0, limit, alpha};      // (gated: 1 SiLU, 2 ReLU, 3 clamped swish, 4 gelu)
   p.sumsq_in = sumsq;
   p.sumsq_units = sumsq_units;
   p.norm_eps = norm_eps;

@@ -20,6 +20,9 @@
 // group): `tok_decay` and `tok_scale` [tokens, H] replace the constant decay and scale the written values,
 // `skip` [H] adds the token's own value to its read-out.
 //
+// `rotate_rows_f32`: the operands of such a scan when q and k are rotated by the token's position: float32 rows q | k | v
+// from the projections, nothing of them rounded after the rotation.
+// `head_norm_gate_out`: y = (o of a head / its root mean square) * act(gate), act SiLU or sigmoid, heads side by side.
 // `linear_attn_out`: y = o / rms(o over all heads) * weight * sigmoid(gate), in the engine's dtype.
 #include "common.cuh"
 
@@ -374,6 +377,183 @@ extern "C" int ll_linear_attn_out(int dtype, void* y, const float* o, const floa
     else
       ll_launch(linear_attn_out_kernel<T, 1>, dim3(num_tokens), dim3(256), 0, stream, (T*)y, o, weight, (const T*)gate,
                 gate_stride, eps, width);
+  });
+  return LL_LAUNCH_RESULT();
+}
+
+// Row t of `out` (float32): H query heads, then H key heads of dk numbers, then the values, at the three offsets.  The first
+// rot_dim numbers of every q and k head turn by angle = float(position) * freq[i], pairs (2i, 2i+1) when `interleaved`,
+// (i, i + rot_dim/2) otherwise: (u, v) -> (u cos a - v sin a, v cos a + u sin a); then q is multiplied by q_scale, k by
+// k_scale.  One block a token; VEC numbers an access (the launcher checked sizes and alignment).
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+rotate_rows_f32_kernel(float* __restrict__ out, long out_stride, int oq, int ok, int ov, const T* __restrict__ proj,
+                       long stride, int iq, int ik, int iv, const int* __restrict__ positions,
+                       const float* __restrict__ freq, int rot_dim, int interleaved, int H, int dk, int vn, float q_scale,
+                       float k_scale) {
+  extern __shared__ float cs[];        // cos [rot_dim / 2], sin [rot_dim / 2]
+  LL_PDL_TRIGGER();
+  LL_PDL_WAIT();
+  const int t = blockIdx.x, tid = threadIdx.x, half = rot_dim >> 1;
+  float* sn = cs + half;
+  const T* row = proj + (size_t)t * stride;
+  float* dst = out + (size_t)t * out_stride;
+  const float pos = (float)positions[t];
+  for (int i = tid; i < half; i += blockDim.x) sincosf(pos * freq[i], &sn[i], &cs[i]);
+  __syncthreads();
+  auto load = [&](const T* p, float* v) {
+    if (VEC == 4) {
+      if (sizeof(T) == 2) {
+        const uint2 u = *reinterpret_cast<const uint2*>(p);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+        v[0] = a.x, v[1 % VEC] = a.y, v[2 % VEC] = b.x, v[3 % VEC] = b.y;
+      } else {
+        const float4 a = *reinterpret_cast<const float4*>(p);
+        v[0] = a.x, v[1 % VEC] = a.y, v[2 % VEC] = a.z, v[3 % VEC] = a.w;
+      }
+    } else {
+      v[0] = to_f32<T>(p[0]);
+    }
+  };
+  auto store = [&](float* p, const float* v) {
+    if (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1 % VEC], v[2 % VEC], v[3 % VEC]);
+    else p[0] = v[0];
+  };
+  const int per = dk / VEC;
+  for (int w = tid; w < 2 * H * per; w += blockDim.x) {
+    const int h = w / per, c = (w - h * per) * VEC;       // q heads, then k heads
+    const bool is_q = h < H;
+    const T* src = row + (is_q ? iq + h * dk : ik + (h - H) * dk);
+    const float scale = is_q ? q_scale : k_scale;
+    float x[VEC], y[VEC];
+    load(src + c, x);
+    if (c < rot_dim) {            // (VEC 4: rot_dim / 2 is a multiple of 4, so the four numbers are on one side)
+      if (interleaved) {
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) y[k] = VEC == 4 ? x[k ^ 1] : to_f32<T>(src[c ^ 1]);
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) {
+          const int i = (c + k) >> 1;
+          x[k] = ((c + k) & 1) ? x[k] * cs[i] + y[k] * sn[i] : x[k] * cs[i] - y[k] * sn[i];
+        }
+      } else {
+        const bool low = c < half;
+        load(src + (low ? c + half : c - half), y);
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) {
+          const int i = (low ? c : c - half) + k;
+          x[k] = low ? x[k] * cs[i] - y[k] * sn[i] : x[k] * cs[i] + y[k] * sn[i];
+        }
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) x[k] *= scale;
+    store(dst + (is_q ? oq + h * dk : ok + (h - H) * dk) + c, x);
+  }
+  for (int w = tid; w < vn / VEC; w += blockDim.x) {
+    float x[VEC];
+    load(row + iv + w * VEC, x);
+    store(dst + ov + w * VEC, x);
+  }
+}
+
+extern "C" int ll_rotate_rows_f32(int dtype, float* out, long out_stride, int oq, int ok, int ov, const void* proj,
+                                  long stride, int iq, int ik, int iv, const int* positions, const float* freq, int rot_dim,
+                                  int interleaved, int H, int dk, int vn, float q_scale, float k_scale, int num_tokens,
+                                  cudaStream_t stream) {
+  if (num_tokens <= 0) return 0;
+  if (H <= 0 || dk <= 0 || vn <= 0 || rot_dim < 0 || rot_dim > dk || (rot_dim & 1) || (rot_dim > 0 && freq == nullptr) ||
+      rot_dim > 8192)
+    return (int)cudaErrorInvalidValue;
+  const int sizes = oq | ok | ov | iq | ik | iv | dk | vn | (rot_dim / 2);
+  const uintptr_t align = dtype == LL_DTYPE_F32 ? 16 : 8;
+  const bool wide = sizes % 4 == 0 && out_stride % 4 == 0 && stride % 4 == 0 && (uintptr_t)out % 16 == 0 &&
+                    (uintptr_t)proj % align == 0;
+  const size_t smem = sizeof(float) * (size_t)rot_dim;
+  LL_DISPATCH_DTYPE(dtype, {
+    if (wide)
+      ll_launch(rotate_rows_f32_kernel<T, 4>, dim3(num_tokens), dim3(256), smem, stream, out, out_stride, oq, ok, ov,
+                (const T*)proj, stride, iq, ik, iv, positions, freq, rot_dim, interleaved, H, dk, vn, q_scale, k_scale);
+    else
+      ll_launch(rotate_rows_f32_kernel<T, 1>, dim3(num_tokens), dim3(256), smem, stream, out, out_stride, oq, ok, ov,
+                (const T*)proj, stride, iq, ik, iv, positions, freq, rot_dim, interleaved, H, dk, vn, q_scale, k_scale);
+  });
+  return LL_LAUNCH_RESULT();
+}
+
+// y[t, h, :] = o[t, h, :] / sqrt(mean(o[t, h, :]^2) + eps) * act(gate[t, h, :]), act 0 SiLU, 1 sigmoid; a warp a (token,
+// head).  VEC = 4: four numbers an access, and heads of up to 32 x 4 x HN_PIECES numbers stay in registers.
+#define HN_PIECES 4
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+head_norm_gate_out_kernel(T* __restrict__ y, const float* __restrict__ o, const T* __restrict__ gate, long gate_stride,
+                          float eps, long pairs, int H, int dv, int act) {
+  LL_PDL_TRIGGER();
+  LL_PDL_WAIT();
+  const long pair = (long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (pair >= pairs) return;
+  const int lane = threadIdx.x & 31;
+  const long t = pair / H;
+  const int h = (int)(pair - t * H);
+  const float* src = o + (size_t)pair * dv;
+  const T* g = gate + (size_t)t * gate_stride + (size_t)h * dv;
+  T* dst = y + (size_t)pair * dv;
+  const bool resident = VEC == 4 && dv <= 32 * 4 * HN_PIECES;
+  float4 x[HN_PIECES];
+  float ss = 0.f;
+  if (resident) {
+#pragma unroll
+    for (int p = 0; p < HN_PIECES; ++p) {
+      const int c = 4 * lane + 128 * p;
+      x[p] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < dv) x[p] = *reinterpret_cast<const float4*>(src + c);
+      ss += (x[p].x * x[p].x + x[p].y * x[p].y) + (x[p].z * x[p].z + x[p].w * x[p].w);
+    }
+  } else {
+    for (int c = lane; c < dv; c += 32) ss = fmaf(src[c], src[c], ss);
+  }
+  const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)dv + eps);
+  auto gated = [&](float v, float z) {
+    const float s = 1.0f / (1.0f + expf(-z));
+    return v * inv * (act == 0 ? z * s : s);
+  };
+  if (resident) {
+#pragma unroll
+    for (int p = 0; p < HN_PIECES; ++p) {
+      const int c = 4 * lane + 128 * p;
+      if (c < dv) {
+        T gv[4], out[4];
+        if (sizeof(T) == 2) *reinterpret_cast<uint2*>(gv) = *reinterpret_cast<const uint2*>(g + c);
+        else *reinterpret_cast<uint4*>(gv) = *reinterpret_cast<const uint4*>(g + c);
+        out[0] = from_f32<T>(gated(x[p].x, to_f32<T>(gv[0])));
+        out[1] = from_f32<T>(gated(x[p].y, to_f32<T>(gv[1])));
+        out[2] = from_f32<T>(gated(x[p].z, to_f32<T>(gv[2])));
+        out[3] = from_f32<T>(gated(x[p].w, to_f32<T>(gv[3])));
+        if (sizeof(T) == 2) *reinterpret_cast<uint2*>(dst + c) = *reinterpret_cast<const uint2*>(out);
+        else *reinterpret_cast<uint4*>(dst + c) = *reinterpret_cast<const uint4*>(out);
+      }
+    }
+  } else {
+    for (int c = lane; c < dv; c += 32) dst[c] = from_f32<T>(gated(src[c], to_f32<T>(g[c])));
+  }
+}
+
+extern "C" int ll_head_norm_gate_out(int dtype, void* y, const float* o, const void* gate, long gate_stride, float eps,
+                                     int num_tokens, int H, int dv, int act, cudaStream_t stream) {
+  if (num_tokens <= 0) return 0;
+  if (H <= 0 || dv <= 0 || act < 0 || act > 1) return (int)cudaErrorInvalidValue;
+  const long pairs = (long)num_tokens * H;
+  const int threads = pairs >= 4096 ? 256 : 64;
+  const dim3 grid((unsigned)((pairs + threads / 32 - 1) / (threads / 32)));
+  const bool wide = dv % 4 == 0 && gate_stride % 4 == 0 && ((uintptr_t)o | (uintptr_t)gate | (uintptr_t)y) % 16 == 0;
+  LL_DISPATCH_DTYPE(dtype, {
+    if (wide)
+      ll_launch(head_norm_gate_out_kernel<T, 4>, grid, dim3(threads), 0, stream, (T*)y, o, (const T*)gate, gate_stride,
+                eps, pairs, H, dv, act);
+    else
+      ll_launch(head_norm_gate_out_kernel<T, 1>, grid, dim3(threads), 0, stream, (T*)y, o, (const T*)gate, gate_stride,
+                eps, pairs, H, dv, act);
   });
   return LL_LAUNCH_RESULT();
 }

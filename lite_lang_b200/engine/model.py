@@ -40,6 +40,7 @@ class PlannedStep:
     layer: int
     caches: Dict[str, PlannedCache]
     add_embedding: bool = False
+    add_row: Optional[int] = None
 
     def _first(self) -> PlannedCache:
         return next(iter(self.caches.values())) if self.caches else PlannedCache(None, 0, False)
@@ -88,6 +89,9 @@ class CausalLM:
             self.blocks.append(block_cls({role: build_part(family, ls.parts[role]) for role, family in roles.items()}))
         self.final_norm = build_part("norm", spec.final_norm)
         self.head = build_part("head", spec.head)
+        self.pass_rows = None if spec.pass_rows is None else build_part("embedding", spec.pass_rows)
+        if self.pass_rows is None and any(rs.add_row is not None for rs in spec.order):
+            raise ValueError("the run order adds rows of 'pass_rows', which the model does not have")
         self.plan, self.cache_groups = self._plan_cache()
         self.dtype: Optional[torch.dtype] = None
         self.device: Optional[torch.device] = None
@@ -123,7 +127,7 @@ class CausalLM:
                     g = len(keys) - 1
                 caches[role] = PlannedCache(g, planes[g], True)
                 planes[g] += 1
-            plan.append(PlannedStep(rs.layer, caches, rs.add_embedding))
+            plan.append(PlannedStep(rs.layer, caches, rs.add_embedding, rs.add_row))
         groups: List[object] = []
         for need, n in zip(keys, planes):
             if isinstance(need, PagedKVNeed):
@@ -139,6 +143,8 @@ class CausalLM:
     # ------------------------------------------------------------------
     def _all_parts(self):
         yield self.embedding
+        if self.pass_rows is not None:
+            yield self.pass_rows
         for b in self.blocks:
             for p in b.parts():
                 yield p
@@ -204,6 +210,8 @@ class CausalLM:
         for ps in self.plan:
             if ps.add_embedding:
                 delta = parts_base.with_extra(delta, h0.float())
+            if ps.add_row is not None:
+                delta = parts_base.with_row(delta, self.pass_rows.row(ps.add_row), n)
             caches = {}
             for role, pc in ps.caches.items():
                 if pc.group is None:

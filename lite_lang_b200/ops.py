@@ -251,11 +251,11 @@ def bias_rotate_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], positions
                 _ptr(v_cache), c_int(page_size), c_long(num_slots), c_int(qkv.shape[0]), _ptr(status), _stream())
 
 
-GATE_ACT = {"silu": 0, "relu": 1, "clamped_swish": 2}
+GATE_ACT = {"silu": 0, "relu": 1, "clamped_swish": 2, "gelu_tanh": 3}
 
 
 class GateAct(NamedTuple):
-    """The activation of a gated product: act(gate) * up with SiLU or ReLU; "clamped_swish": with a = min(gate, limit)
+    """The activation of a gated product: act(gate) * up with SiLU, ReLU or the tanh form of GELU; "clamped_swish": with a = min(gate, limit)
     and c = clamp(up, -limit, limit), a * sigmoid(alpha a) * (c + 1)."""
     kind: str
     limit: float = 0.0
@@ -515,13 +515,16 @@ def attn_prefill_tc(out: torch.Tensor, q: torch.Tensor, q_stride: int, k_cache: 
                     block_table: torch.Tensor, cu_q: torch.Tensor, ctx_len: torch.Tensor, req_slot: torch.Tensor,
                     num_entries: int, row_blocks: int, num_heads: int, num_kv_heads: int, head_dim: int,
                     page_size: int, window: Optional[int], scale: float, status: Optional[torch.Tensor],
-                    nsplit: Optional[int] = None, split_len: int = 8, gate: Optional[torch.Tensor] = None) -> None:
+                    nsplit: Optional[int] = None, split_len: int = 8, gate: Optional[torch.Tensor] = None,
+                    pairs: Optional["MapPairs"] = None) -> None:
     """Paged attention for portions of prompts on the tcgen05 tensor cores (TMA loads, S and O in tensor
     memory).  ``row_blocks`` from ``attn_prefill_tc_blocks``.  Otherwise as ``attn_prefill``.
     ``nsplit`` (1, 2, 4, 8; default: by the size of the step): the keys of a row block are split over up to that
     many CTAs of about ``split_len`` blocks of 64 keys each (``attn_prefill_tc_plan`` chooses both), which merge
     through scratch memory kept by this module (grown when needed, never shrunk).
-    ``gate`` (bfloat16 [tokens, num_heads], any row stride): every head's output times the sigmoid of its gate."""
+    ``gate`` (bfloat16 [tokens, num_heads], any row stride): every head's output times the sigmoid of its gate.
+    ``pairs``: the query heads are pairs of score maps, and half as many heads come out (and have gates)."""
+    heads_out = num_heads if pairs is None else num_heads // 2
     _need_cuda(out, q, k_cache, v_cache, block_table, cu_q, ctx_len, req_slot, gate)
     for t, nm in ((block_table, "block_table"), (cu_q, "cu_q"), (ctx_len, "ctx_len"), (req_slot, "req_slot")):
         _i32(t, nm)
@@ -530,7 +533,7 @@ def attn_prefill_tc(out: torch.Tensor, q: torch.Tensor, q_stride: int, k_cache: 
           f"not {q.dtype}, {head_dim}, {page_size}")
     _need(out.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and v_cache.dtype == torch.bfloat16,
           "attn_prefill_tc: dtypes differ")
-    _need(out.stride(1) == 1 and out.shape[1] == num_heads * head_dim and out.stride(0) % 8 == 0,
+    _need(out.stride(1) == 1 and out.shape[1] == heads_out * head_dim and out.stride(0) % 8 == 0,
           "attn_prefill_tc: out")
     _need(q.stride(1) == 1 and q.shape[1] >= num_heads * head_dim and q.stride(0) == q_stride, "attn_prefill_tc: q")
     _need(k_cache.is_contiguous() and v_cache.is_contiguous(), "cache plane must be contiguous")
@@ -556,7 +559,13 @@ def attn_prefill_tc(out: torch.Tensor, q: torch.Tensor, q_stride: int, k_cache: 
             c_int(max(1, int(split_len))), _ptr(scratch), _ptr(counters))
     if gate is not None:
         _need(gate.dtype == torch.bfloat16 and gate.dim() == 2 and gate.shape[0] == q.shape[0]
-              and gate.shape[1] == num_heads and gate.stride(1) == 1, "attn_prefill_tc: gate is bfloat16 [tokens, heads]")
+              and gate.shape[1] == heads_out and gate.stride(1) == 1, "attn_prefill_tc: gate is bfloat16 [tokens, heads]")
+    if pairs is not None:
+        load_library("attn_tc").call("ll_attn_prefill_tc_pairs", *args, _ptr(gate),
+                                     c_long(0 if gate is None else gate.stride(0)), c_float(pairs.weight),
+                                     c_float(pairs.post), c_float(pairs.eps), _ptr(status), _stream())
+        return
+    if gate is not None:
         load_library("attn_tc").call("ll_attn_prefill_tc_gated", *args, _ptr(gate), c_long(gate.stride(0)), _ptr(status),
                                      _stream())
         return
@@ -1638,6 +1647,100 @@ def linear_attn_out(y: torch.Tensor, o: torch.Tensor, weight: torch.Tensor, gate
 # --------------------------------------------------------------------------
 # a norm on the sublayer's output, a plain feed-forward's activation, scaled logits
 # --------------------------------------------------------------------------
+def sandwich_norm(out: Optional[torch.Tensor], residual: torch.Tensor, y: Optional[torch.Tensor],
+                  y_weight: Optional[torch.Tensor], y_eps: float, add: Optional[torch.Tensor],
+                  weight: Optional[torch.Tensor], eps: float, rows: Optional[torch.Tensor] = None) -> None:
+    """residual (float32) += y / sqrt(mean(y^2) + y_eps) * y_weight + add (written back unless ``rows`` selects rows); out =
+    residual / sqrt(mean^2 + eps) * weight, or without ``weight`` the residual itself, in ``out``'s dtype.  ``y``: [tokens,
+    hidden] of ``out``'s dtype, or float32 partial sums [parts, tokens, hidden]; ``add`` float32 [hidden], one row for all
+    tokens.  ``y``, ``add`` and ``out`` may be None."""
+    _need_cuda(out, residual, y, y_weight, add, weight, rows)
+    for t, nm in ((residual, "residual"), (y_weight, "output norm weight"), (add, "add"), (weight, "norm weight")):
+        _f32(t, nm)
+    _i32(rows, "rows")
+    n_all, W = residual.shape
+    n = n_all if rows is None else rows.numel()
+    _need(residual.is_contiguous(), "sandwich_norm: residual rows")
+    for t in (y_weight, add, weight):
+        _need(t is None or t.numel() == W, "sandwich_norm: a weight has one number a channel")
+    _need(out is None or (out.is_contiguous() and tuple(out.shape) == (n, W)), "sandwich_norm: out")
+    partial, parts, part_stride = None, 0, 0
+    dt = 0 if out is None else _dtype_code(out)
+    if y is not None:
+        _need(y_weight is not None and y.is_contiguous(), "sandwich_norm: y and its weight")
+        if y.dim() == 3:
+            _need(y.dtype == torch.float32 and tuple(y.shape[1:]) == (n_all, W), "sandwich_norm: partial sums")
+            partial, parts, part_stride, y = y, y.shape[0], n_all * W, None
+        else:
+            _need(tuple(y.shape) == (n_all, W) and (out is None or y.dtype == out.dtype), "sandwich_norm: y")
+            dt = _dtype_code(y)
+    load_library("sandwich").call(
+        "ll_sandwich_norm", c_int(dt), _ptr(out), _ptr(residual), _ptr(y), _ptr(partial), c_int(parts), c_long(part_stride),
+        _ptr(y_weight), c_float(y_eps), _ptr(add), _ptr(weight), c_float(eps), c_int(n), c_int(W), _ptr(rows),
+        c_int(1 if rows is None and (y is not None or partial is not None or add is not None) else 0), _stream())
+
+
+def embed_norm(out: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, weight: torch.Tensor, eps: float,
+               status: Optional[torch.Tensor]) -> None:
+    """out[t] = RMS norm of table[ids[t]] times ``weight`` as float32 rows."""
+    _need_cuda(out, table, ids, weight)
+    _i32(ids, "ids")
+    _f32(out, "out")
+    _f32(weight, "weight")
+    _need(table.is_contiguous() and out.is_contiguous() and out.shape[1] == table.shape[1] == weight.numel()
+          and out.shape[0] >= ids.numel(), "embed_norm: shapes")
+    load_library("sandwich").call(
+        "ll_embed_norm", c_int(_dtype_code(table)), _ptr(out), _ptr(table), _ptr(ids), _ptr(weight), c_float(eps),
+        c_int(ids.numel()), c_int(table.shape[1]), c_int(table.shape[0]), _ptr(status), _stream())
+
+
+def token_side_act(g: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, status: Optional[torch.Tensor]) -> None:
+    """g[t] <- gelu_tanh(g[t]) * table[ids[t]] in place; ``table`` may be a slice of columns of a wider table."""
+    _need_cuda(g, table, ids)
+    _i32(ids, "ids")
+    _need(g.dim() == 2 and g.stride(1) == 1 and table.stride(1) == 1 and table.dtype == g.dtype
+          and table.shape[1] == g.shape[1] and ids.numel() >= g.shape[0], "token_side_act: shapes")
+    load_library("sandwich").call(
+        "ll_token_side_act", c_int(_dtype_code(g)), _ptr(g), c_long(g.stride(0)), _ptr(table), c_long(table.stride(0)),
+        _ptr(ids), c_int(g.shape[0]), c_int(g.shape[1]), c_int(table.shape[0]), c_int(sm_count(g.device)), _ptr(status),
+        _stream())
+
+
+def rotate_rows_f32(out: torch.Tensor, out_offsets, proj: torch.Tensor, offsets, positions: torch.Tensor,
+                    freq: Optional[torch.Tensor], interleaved: bool, H: int, dk: int, v_width: int, q_scale: float,
+                    k_scale: float) -> None:
+    """float32 rows q | k | v (``out_offsets``) from the projections (``offsets``), q and k heads rotated by the token's
+    position (angles made in the kernel) and then multiplied by a constant each."""
+    _need_cuda(out, proj, positions, freq)
+    _f32(out, "out")
+    _f32(freq, "freq")
+    _i32(positions, "positions")
+    _need(out.stride(1) == 1 and proj.stride(1) == 1 and out.shape[0] == proj.shape[0], "rotate_rows_f32: rows")
+    for offs, t in ((out_offsets, out), (offsets, proj)):
+        _need(max(offs[0] + H * dk, offs[1] + H * dk, offs[2] + v_width) <= t.shape[1], "rotate_rows_f32: columns")
+    rot = 0 if freq is None else 2 * freq.numel()
+    _need(rot <= dk, "rotate_rows_f32: rot_dim <= dk")
+    load_library("linear_attn").call(
+        "ll_rotate_rows_f32", c_int(_dtype_code(proj)), _ptr(out), c_long(out.stride(0)), *(c_int(o) for o in out_offsets),
+        _ptr(proj), c_long(proj.stride(0)), *(c_int(o) for o in offsets), _ptr(positions), _ptr(freq), c_int(rot),
+        c_int(1 if interleaved else 0), c_int(H), c_int(dk), c_int(v_width), c_float(q_scale), c_float(k_scale),
+        c_int(proj.shape[0]), _stream())
+
+
+HEAD_GATE_ACT = {"silu": 0, "sigmoid": 1}
+
+
+def head_norm_gate_out(y: torch.Tensor, o: torch.Tensor, gate: torch.Tensor, eps: float, H: int, dv: int, act: str) -> None:
+    """y = every head of ``o`` (float32 [tokens, H * dv]) divided by its root mean square, times act(gate)."""
+    _need_cuda(y, o, gate)
+    _f32(o, "o")
+    _need(y.is_contiguous() and o.is_contiguous() and tuple(y.shape) == tuple(o.shape) == (y.shape[0], H * dv)
+          and tuple(gate.shape) == tuple(y.shape) and gate.dtype == y.dtype and gate.stride(1) == 1, "head_norm_gate_out")
+    load_library("linear_attn").call(
+        "ll_head_norm_gate_out", c_int(_dtype_code(y)), _ptr(y), _ptr(o), _ptr(gate), c_long(gate.stride(0)), c_float(eps),
+        c_int(y.shape[0]), c_int(H), c_int(dv), c_int(HEAD_GATE_ACT[act]), _stream())
+
+
 def layernorm_into_residual(residual: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: float,
                             copy: Optional[torch.Tensor]) -> None:
     """residual (float32) += layer norm of y times ``weight``; ``copy`` (optional) receives the new residual rows
@@ -1712,8 +1815,22 @@ def scale_logits(logits: torch.Tensor, factor: float) -> None:
 # --------------------------------------------------------------------------
 # attention with normalised q, k, v and shaped scores
 # --------------------------------------------------------------------------
-QK_NORM = {None: 0, "none": 0, "head_unit": 1, "projection": 2}
+QK_NORM = {None: 0, "none": 0, "head_unit": 1, "projection": 2, "head": 3}
 ATTN_MASK = {"causal": 0, "window": 1, "chunk": 2}
+
+
+class MapPairs(NamedTuple):
+    """Neighbouring query heads 2a and 2a + 1 of an attention are two score maps over the same keys and values and come
+    out as one head: z = o_even - ``weight`` * o_odd, then z / sqrt(mean(z^2) + ``eps``) * ``post`` (before a gate)."""
+    weight: float
+    post: float
+    eps: float
+
+
+def _pair_args(pairs: Optional[MapPairs]):
+    if pairs is None:
+        return c_int(0), c_float(0.0), c_float(0.0), c_float(0.0)
+    return c_int(1), c_float(pairs.weight), c_float(pairs.post), c_float(pairs.eps)
 
 
 def qkv_norm_rotate_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], positions: torch.Tensor,
@@ -1723,15 +1840,24 @@ def qkv_norm_rotate_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], posit
                           eps: float, slot_map: Optional[torch.Tensor], k_cache: Optional[torch.Tensor],
                           v_cache: Optional[torch.Tensor], page_size: int, status: Optional[torch.Tensor],
                           head_mix: Optional[torch.Tensor] = None, mix_temperature: Optional[torch.Tensor] = None,
-                          mixed_q: Optional[torch.Tensor] = None) -> None:
+                          mixed_q: Optional[torch.Tensor] = None, paired_q: Optional[torch.Tensor] = None) -> None:
     """Bias, the norms of q, k and v (``qk_norm``: "projection": an RMS norm with weights over all of q and all of
     k before the rotation; "head_unit": every head divided by its root mean square after it; ``value_norm``: the
-    same for every value head), the rotation by angles made in the kernel (cos and sin times ``amplitude``), and
+    same for every value head; "head": every q and k head through an RMS norm before the rotation, one weight of head_dim
+    numbers for all q heads and one for all k heads), the rotation by angles made in the kernel (cos and sin times ``amplitude``), and
     the store of k and v.  In place on the first (nh + nkv) * head_dim + nkv * value_head_dim columns of ``qkv``.
     With ``head_mix`` [nh, nh] and ``mixed_q`` [tokens, nh * nkv * head_dim] also the queries of an attention that
-    mixes its heads' scores, as one wider query a head over all kv heads' keys side by side (``attn_shaped``)."""
+    mixes its heads' scores, as one wider query a head over all kv heads' keys side by side (``attn_shaped``).
+    With ``paired_q`` [tokens, nh * 2 * head_dim] (an attention of ``MapPairs``) q and k heads come in neighbouring pairs and
+    there are nkv / 2 value heads: a cached key row is a pair's two parts side by side, and ``paired_q`` receives the
+    queries, each beside zeros in the place of the other map's part."""
     _need_cuda(qkv, bias, positions, freq, q_weight, k_weight, slot_map, k_cache, v_cache, head_mix, mix_temperature,
-               mixed_q)
+               mixed_q, paired_q)
+    maps = 1 if paired_q is None else 2
+    num_value_heads = num_kv_heads // maps
+    _need(num_kv_heads % maps == 0 and num_heads % maps == 0, "paired heads come in twos")
+    _need(paired_q is None or (paired_q.dtype == qkv.dtype and paired_q.is_contiguous() and mixed_q is None
+                               and tuple(paired_q.shape) == (qkv.shape[0], num_heads * 2 * head_dim)), "paired_q shape")
     _f32(head_mix, "head_mix")
     _f32(mix_temperature, "mix_temperature")
     if mixed_q is not None:
@@ -1743,10 +1869,13 @@ def qkv_norm_rotate_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], posit
         _f32(t, nm)
     _i32(positions, "positions")
     _i32(slot_map, "slot_map")
-    width = (num_heads + num_kv_heads) * head_dim + num_kv_heads * value_head_dim
-    _need(qkv.dim() == 2 and qkv.shape[1] >= width and qkv.stride(1) == 1, "qkv must be [tokens, >= (nh+nkv)*hd + nkv*vd]")
+    width = (num_heads + num_kv_heads) * head_dim + num_value_heads * value_head_dim
+    _need(qkv.dim() == 2 and qkv.shape[1] >= width and qkv.stride(1) == 1, "qkv must be [tokens, >= (nh+nkv)*hd + nv*vd]")
     _need(bias is None or bias.numel() == width, "bias size")
     mode = QK_NORM[qk_norm]
+    if mode == 3:
+        _need(q_weight is not None and q_weight.numel() == head_dim and k_weight is not None
+              and k_weight.numel() == head_dim, "head norm: a weight of head_dim numbers for q and one for k")
     if mode == 2:
         _need(q_weight is not None and q_weight.numel() == num_heads * head_dim and k_weight is not None
               and k_weight.numel() == num_kv_heads * head_dim, "projection norm: weights over all of q and all of k")
@@ -1757,8 +1886,8 @@ def qkv_norm_rotate_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], posit
         _need(k_cache is not None and v_cache is not None, "store needs the cache plane")
         _need(k_cache.dtype == qkv.dtype and v_cache.dtype == qkv.dtype, "cache dtype differs from activations")
         _need(k_cache.is_contiguous() and v_cache.is_contiguous(), "cache plane must be contiguous")
-        _need(tuple(k_cache.shape[1:]) == (num_kv_heads, page_size, head_dim)
-              and tuple(v_cache.shape[1:]) == (num_kv_heads, page_size, value_head_dim), "cache plane shape")
+        _need(tuple(k_cache.shape[1:]) == (num_value_heads, page_size, maps * head_dim)
+              and tuple(v_cache.shape[1:]) == (num_value_heads, page_size, value_head_dim), "cache plane shape")
         num_slots = k_cache.shape[0] * page_size
     load_library("attn_mod").call(
         "ll_qkv_norm_rotate_store", c_int(_dtype_code(qkv)), _ptr(qkv), c_long(qkv.stride(0)), _ptr(bias),
@@ -1766,7 +1895,7 @@ def qkv_norm_rotate_store(qkv: torch.Tensor, bias: Optional[torch.Tensor], posit
         c_int(num_heads), c_int(num_kv_heads), c_int(head_dim), c_int(value_head_dim), c_int(mode), _ptr(q_weight),
         _ptr(k_weight), c_int(1 if value_norm else 0), c_float(eps), _ptr(slot_map), _ptr(k_cache), _ptr(v_cache),
         c_int(page_size), c_long(num_slots), c_int(qkv.shape[0]), _ptr(head_mix if mixed_q is not None else None),
-        _ptr(mix_temperature), _ptr(mixed_q), _ptr(status), _stream())
+        _ptr(mix_temperature), _ptr(mixed_q), c_int(maps), _ptr(paired_q), _ptr(status), _stream())
 
 
 def attn_shaped_supported(dtype: torch.dtype, num_kv_heads: int, head_dim: int, value_head_dim: int, page_size: int,
@@ -1794,7 +1923,7 @@ def attn_shaped(out: torch.Tensor, q: torch.Tensor, q_stride: int, mixed: bool, 
                 keep_first: int = 0, softcap: Optional[float] = None,
                 query_temperature: Optional[Tuple[float, int]] = None, gate_channels: bool = False,
                 out_scale: float = 1.0,
-                distance_slope: Optional[torch.Tensor] = None) -> None:
+                distance_slope: Optional[torch.Tensor] = None, pairs: Optional[MapPairs] = None) -> None:
     """Tensor-core paged attention (bfloat16) with shaped scores: the mechanisms of ``attention_modulated`` for
     head sizes 64 and 128.  ``q``: the projection's rows (head h at h * head_dim), or with ``mixed`` the wider
     queries that ``qkv_norm_rotate_store`` leaves for mixed heads (then ``temperature`` is inside them).
@@ -1802,7 +1931,8 @@ def attn_shaped(out: torch.Tensor, q: torch.Tensor, q_stride: int, mixed: bool, 
     keys, each a CTA, joined by a second kernel; nsplit * span must cover the stages any token sees (kept first
     tokens' stages before the window's are walked by the first part besides).  ``sink_values``, ``distance_bias``,
     ``keep_first``, ``softcap``, ``query_temperature``, ``gate_channels``, ``out_scale`` and ``distance_slope`` are those
-    of ``attention_modulated``.  Launches one kernel, two with ``nsplit`` > 1."""
+    of ``attention_modulated``, and so are ``pairs``.  Launches one kernel, two with ``nsplit`` > 1."""
+    heads_out = num_heads if pairs is None else num_heads // 2
     _need_cuda(out, q, gate, temperature, k_cache, v_cache, block_table, cu_q, ctx_len, req_slot, sink_values,
                distance_bias)
     _need_cuda(distance_slope)
@@ -1821,7 +1951,7 @@ def attn_shaped(out: torch.Tensor, q: torch.Tensor, q_stride: int, mixed: bool, 
           "attn_shaped takes bfloat16, head sizes 64 and 128 and pages of a multiple of 16 tokens")
     _need(out.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and v_cache.dtype == torch.bfloat16,
           "attn_shaped: dtypes differ")
-    _need(out.stride(1) == 1 and out.shape[1] == num_heads * value_head_dim and out.stride(0) % 8 == 0,
+    _need(out.stride(1) == 1 and out.shape[1] == heads_out * value_head_dim and out.stride(0) % 8 == 0,
           "attn_shaped: out")
     _need(k_cache.is_contiguous() and v_cache.is_contiguous(), "cache plane must be contiguous")
     _need(tuple(k_cache.shape[1:]) == (num_kv_heads, page_size, head_dim)
@@ -1830,7 +1960,7 @@ def attn_shaped(out: torch.Tensor, q: torch.Tensor, q_stride: int, mixed: bool, 
           "attn_shaped: entry arrays too short")
     _need(temperature is None or temperature.numel() == num_heads, "temperature: a number a head")
     _need(gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1
-                           and gate.shape[1] == (num_heads * value_head_dim if gate_channels else num_heads)),
+                           and gate.shape[1] == (heads_out * value_head_dim if gate_channels else heads_out)),
           "gate: [tokens, heads] rows (or a number a channel)")
     _need(mask == "causal" or (mask_size or 0) > 0, "a window or chunks need a size")
     part = None
@@ -1847,7 +1977,7 @@ def attn_shaped(out: torch.Tensor, q: torch.Tensor, q_stride: int, mixed: bool, 
         _ptr(status), _ptr(sink_values), _ptr(distance_bias),
         c_int(0 if distance_bias is None else distance_bias.shape[0]), c_int(int(keep_first or 0)),
         c_float(float(softcap or 0.0)), c_float(qt_coef), c_int(qt_every), c_int(1 if gate_channels else 0),
-        c_float(out_scale), _ptr(distance_slope), _stream())
+        c_float(out_scale), _ptr(distance_slope), *_pair_args(pairs), _stream())
 
 
 def attention_modulated(out: torch.Tensor, q: torch.Tensor, q_stride: int, gate: Optional[torch.Tensor],
@@ -1860,7 +1990,7 @@ def attention_modulated(out: torch.Tensor, q: torch.Tensor, q_stride: int, gate:
                         distance_bias: Optional[torch.Tensor] = None, keep_first: int = 0,
                         softcap: Optional[float] = None, query_temperature: Optional[Tuple[float, int]] = None,
                         gate_channels: bool = False, out_scale: float = 1.0,
-                        distance_slope: Optional[torch.Tensor] = None) -> None:
+                        distance_slope: Optional[torch.Tensor] = None, pairs: Optional[MapPairs] = None) -> None:
     """Attention of every new token over its request's cached keys with shaped scores (any sizes, both dtypes):
     a number a head on the scores (``temperature``), the heads' scores mixed by ``head_mix`` [nh, nh], a window
     or chunks (``mask``, ``mask_size``), one more key of score 0 without a value (``sink``), a sigmoid gate a
@@ -1871,7 +2001,9 @@ def attention_modulated(out: torch.Tensor, q: torch.Tensor, q_stride: int, gate:
     ``query_temperature`` (coef, every): the scores of the query at position p times
     1 + coef ln(floor((p + 1) / every) + 1).  ``gate_channels``: ``gate`` is [tokens, nh * vd], a gate a channel.
     ``out_scale``: a constant on the output, applied before its one rounding.  ``distance_slope`` float32 [nh]: a key n
-    positions back has slope_h * n taken off its score (after the cap)."""
+    positions back has slope_h * n taken off its score (after the cap).  ``pairs``: the query heads are pairs of score maps,
+    and half as many heads come out (and have gates)."""
+    heads_out = num_heads if pairs is None else num_heads // 2
     _need_cuda(out, q, gate, k_cache, v_cache, block_table, token_req, req_slot, positions, temperature, head_mix,
                sink_values, distance_bias)
     _need_cuda(distance_slope)
@@ -1889,14 +2021,14 @@ def attention_modulated(out: torch.Tensor, q: torch.Tensor, q_stride: int, gate:
     _f32(head_mix, "head_mix")
     _need(num_heads % num_kv_heads == 0, "num_heads must be a multiple of num_kv_heads")
     _need(out.dtype == q.dtype == k_cache.dtype == v_cache.dtype, "attention: dtypes differ")
-    _need(out.stride(1) == 1 and out.shape[1] == num_heads * value_head_dim, "attention: out shape")
+    _need(out.stride(1) == 1 and out.shape[1] == heads_out * value_head_dim, "attention: out shape")
     _need(k_cache.is_contiguous() and v_cache.is_contiguous(), "cache plane must be contiguous")
     _need(tuple(k_cache.shape[1:]) == (num_kv_heads, page_size, head_dim)
           and tuple(v_cache.shape[1:]) == (num_kv_heads, page_size, value_head_dim), "cache plane shape")
     _need(temperature is None or temperature.numel() == num_heads, "temperature: a number a head")
     _need(head_mix is None or tuple(head_mix.shape) == (num_heads, num_heads), "head_mix is [heads, heads]")
     _need(gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1
-                           and gate.shape[1] == (num_heads * value_head_dim if gate_channels else num_heads)),
+                           and gate.shape[1] == (heads_out * value_head_dim if gate_channels else heads_out)),
           "gate: a number a head (or a channel) and token, rows of the projection's dtype")
     qt_coef, qt_every = (0.0, 0) if query_temperature is None else (float(query_temperature[0]), int(query_temperature[1]))
     load_library("attn_mod").call(
@@ -1909,7 +2041,7 @@ def attention_modulated(out: torch.Tensor, q: torch.Tensor, q_stride: int, gate:
         c_int(0 if distance_bias is None else distance_bias.shape[0]), c_int(int(keep_first or 0)),
         c_float(float(softcap or 0.0)), c_float(qt_coef), c_int(qt_every),
         c_long(0 if gate is None else gate.stride(0)), c_int(1 if gate_channels else 0), c_float(out_scale),
-        _ptr(distance_slope), _stream())
+        _ptr(distance_slope), *_pair_args(pairs), _stream())
 
 
 # --------------------------------------------------------------------------

@@ -224,19 +224,51 @@ class Pending(NamedTuple):
     extra: Optional[torch.Tensor] = None     # float32 [tokens, hidden]
 
 
+class NormedOutput(NamedTuple):
+    """A sublayer's output whose own norm is still to be taken: y / sqrt(mean(y^2) + eps) * weight (+ ``row``, one float32
+    row for all tokens) is what the residual gains.  The norm that reads the residual next takes it in its pass."""
+    y: Optional[torch.Tensor]                # [tokens, hidden], or float32 partial sums [parts, tokens, hidden]; None: the row alone
+    weight: Optional[torch.Tensor] = None    # float32 [hidden]
+    eps: float = 0.0
+    row: Optional[torch.Tensor] = None       # float32 [hidden]
+
+    def gain(self) -> Optional[torch.Tensor]:
+        """What it adds to the residual, as float32 rows (for readers without a fused pass)."""
+        if self.y is None:
+            return None if self.row is None else self.row[None, :]
+        y = self.y.sum(0) if self.y.dim() == 3 else self.y.float()
+        out = y * torch.rsqrt((y * y).mean(-1, keepdim=True) + self.eps) * self.weight
+        return out if self.row is None else out + self.row
+
+
+def with_row(delta, row: torch.Tensor, tokens: int):
+    """The pending output ``delta`` and one float32 ``row`` [hidden] for every token besides."""
+    if delta is None or isinstance(delta, ResidualCopy):
+        return NormedOutput(None, row=row)
+    if isinstance(delta, NormedOutput):
+        return delta._replace(row=row if delta.row is None else delta.row + row)
+    return with_extra(delta, row[None, :].expand(tokens, -1).contiguous())
+
+
 def with_extra(delta, extra: torch.Tensor) -> Pending:
     """The pending output ``delta`` and ``extra`` rows besides."""
     if delta is None or isinstance(delta, ResidualCopy):
         return Pending(extra=extra)
     if isinstance(delta, Pending):
         return delta._replace(extra=extra if delta.extra is None else delta.extra + extra)
+    if isinstance(delta, NormedOutput):
+        gain = delta.gain()
+        return Pending(extra=extra if gain is None else extra + gain)
     if isinstance(delta, torch.Tensor):
         return Pending(y=delta, extra=extra)
     raise TypeError(f"rows cannot be added to a pending {type(delta).__name__}")
 
 
 def settled(delta, dtype: torch.dtype):
-    """A ``Pending`` as one tensor of ``dtype`` (None if nothing is pending); anything else as it is."""
+    """A ``Pending`` (or a ``NormedOutput``) as one tensor of ``dtype`` (None if nothing is pending); anything else as it is."""
+    if isinstance(delta, NormedOutput):
+        gain = delta.gain()
+        return None if gain is None else gain.to(dtype)
     if not isinstance(delta, Pending):
         return delta
     total = None if delta.y is None else (delta.y.sum(0) if delta.y.dim() == 3 else delta.y.float())

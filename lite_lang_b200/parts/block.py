@@ -106,6 +106,50 @@ class ParallelMixerOnlyBlock(Block):
         return h, self.mixer.forward(x, step, caches["mixer"])
 
 
+class SandwichBlock(Block):
+    """A norm before and a norm behind every sublayer: h += N1b(mixer(N1(h))); h += N2b(feed_forward(N2(h))).  An output
+    norm, the residual sum and the input norm after it are one pass (``NormedOutput``)."""
+
+    roles = {"mixer_norm": "norm", "mixer": "mixer", "mixer_out_norm": "norm",
+             "feed_forward_norm": "norm", "feed_forward": "feed_forward", "feed_forward_out_norm": "norm"}
+
+    def sublayers(self, h, delta, step, caches):
+        """What is pending after the layer's sublayers."""
+        x = self.mixer_norm.add_forward(h, delta)
+        p = self.mixer_out_norm.pending(self.mixer.forward(x, step, caches["mixer"]))
+        if "feed_forward" not in self.roles:
+            return p
+        x = self.feed_forward_norm.add_forward(h, p)
+        return self.feed_forward_out_norm.pending(self.feed_forward.forward(x, step))
+
+    def forward(self, h, delta, step, caches):
+        return h, self.sublayers(h, delta, step, caches)
+
+
+class SandwichMixerOnlyBlock(SandwichBlock):
+    """The same for a layer without a feed-forward."""
+
+    roles = {"mixer_norm": "norm", "mixer": "mixer", "mixer_out_norm": "norm"}
+
+
+class SandwichTokenSideBlock(SandwichBlock):
+    """The same with a third sublayer that reads the residual itself (no norm before it) and the step's token ids:
+    h += N3(side(h, tokens))."""
+
+    roles = {**SandwichBlock.roles, "token_side": "feed_forward", "token_side_out_norm": "norm"}
+
+    def forward(self, h, delta, step, caches):
+        p = self.sublayers(h, delta, step, caches)
+        x = self.token_side_out_norm.apply(h, p, self.token_side.dtype)
+        return h, self.token_side_out_norm.pending(self.token_side.forward(x, step))
+
+
+class SandwichTokenSideMixerOnlyBlock(SandwichTokenSideBlock):
+    """The same for a layer without a feed-forward."""
+
+    roles = {**SandwichMixerOnlyBlock.roles, "token_side": "feed_forward", "token_side_out_norm": "norm"}
+
+
 class OutputNormBlock(Block):
     """Norm on the sublayers' outputs: h += norm(mixer(h)); h += norm(feed_forward(h)).  The sublayers read the
     float32 residual stream itself, rounded to the engine's dtype; that copy is made by the norm's pass over the
@@ -145,5 +189,9 @@ register_part("block", "pre_norm_conv", PreNormConvBlock)
 register_part("block", "pre_norm_conv_mixer_only", PreNormConvMixerOnlyBlock)
 register_part("block", "output_norm", OutputNormBlock)
 register_part("block", "output_norm_mixer_only", OutputNormMixerOnlyBlock)
+register_part("block", "sandwich", SandwichBlock)
+register_part("block", "sandwich_mixer_only", SandwichMixerOnlyBlock)
+register_part("block", "sandwich_token_side", SandwichTokenSideBlock)
+register_part("block", "sandwich_token_side_mixer_only", SandwichTokenSideMixerOnlyBlock)
 register_part("block", "parallel", ParallelBlock)
 register_part("block", "parallel_mixer_only", ParallelMixerOnlyBlock)

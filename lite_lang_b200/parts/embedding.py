@@ -37,15 +37,27 @@ class TokenEmbedding(Part):
             raise ValueError(f"token_embedding: residual {self.residual!r} is neither 'compute' nor 'float32'")
         if self.residual == "compute" and self.scale != 1.0:
             raise ValueError("token_embedding: a scale is built for a float32 residual stream only")
+        # ``norm``: {"tensor", "eps"}: the rows go through an RMS norm with that weight (a float32 residual of one stream)
+        self.norm = None if not spec.params.get("norm") else dict(spec.params["norm"])
+        if self.norm is not None and (self.residual != "float32" or self.streams != 1 or self.scale != 1.0):
+            raise ValueError("token_embedding: a norm is built for an unscaled float32 residual of one stream")
         self.weight: Optional[torch.Tensor] = None
+        self.norm_weight: Optional[torch.Tensor] = None
 
     def tensors(self) -> Dict[str, TensorDecl]:
-        return {self.tensor: TensorDecl((self.vocab_size, self.hidden_size))}
+        d = {self.tensor: TensorDecl((self.vocab_size, self.hidden_size))}
+        if self.norm is not None:
+            d[str(self.norm["tensor"])] = TensorDecl((self.hidden_size,), "norm")
+        return d
 
     def load(self, fetch, dtype, device) -> None:
         self.weight = fetch(self.tensor).to(dtype).to(device).contiguous()
+        if self.norm is not None:
+            self.norm_weight = fetch(str(self.norm["tensor"])).to(torch.float32).to(device).contiguous()
 
     def kernel_libraries(self):
+        if self.norm is not None:
+            return ("core", "sandwich")
         return ("core", "streams") if self.streams != 1 else ("core",)
 
     def forward(self, token_ids: torch.Tensor, num_tokens: int, status) -> torch.Tensor:
@@ -56,11 +68,37 @@ class TokenEmbedding(Part):
             return out
         if self.residual == "float32":
             out = torch.empty((num_tokens, self.hidden_size), dtype=torch.float32, device=self.weight.device)
+            if self.norm is not None:
+                ops.embed_norm(out, self.weight, token_ids[:num_tokens], self.norm_weight, float(self.norm["eps"]), status)
+                return out
             ops.embed_scaled_f32(out, self.weight, token_ids[:num_tokens], self.scale, status)
             return out
         out = torch.empty((num_tokens, self.hidden_size), dtype=self.weight.dtype, device=self.weight.device)
         ops.embed_gather(out, self.weight, token_ids[:num_tokens], status)
         return out
+
+
+class PassRows(Part):
+    """A row for every pass of a range of layers that runs several times, added to the residual of all tokens right before
+    the pass (``RunStep.add_row`` names the row).  float32 on the device."""
+
+    kind_family = "embedding"
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.rows = int(spec.params["rows"])
+        self.hidden_size = int(spec.params["hidden_size"])
+        self.tensor = str(spec.params.get("tensor", "weight"))
+        self.table: Optional[torch.Tensor] = None
+
+    def tensors(self) -> Dict[str, TensorDecl]:
+        return {self.tensor: TensorDecl((self.rows, self.hidden_size), "bias")}
+
+    def load(self, fetch, dtype, device) -> None:
+        self.table = fetch(self.tensor).to(torch.float32).to(device).contiguous()
+
+    def row(self, i: int) -> torch.Tensor:
+        return self.table[i]
 
 
 class LMHead(Part):
@@ -100,4 +138,5 @@ class LMHead(Part):
 
 
 register_part("embedding", "token_embedding", TokenEmbedding)
+register_part("embedding", "pass_rows", PassRows)
 register_part("head", "lm_head", LMHead)

@@ -27,7 +27,7 @@ class GatedMLP(FeedForward):
         if act not in ops.GATE_ACT:
             raise ValueError(f"gated_mlp: activation {act!r} is not built ({', '.join(ops.GATE_ACT)})")
         # "clamped_swish": with a = min(gate x, ``limit``) and c = clamp(up x, -limit, limit), down(a sigmoid(``swish_alpha``
-        # a) (c + 1))
+        # a) (c + 1)); "gelu_tanh": the tanh form of GELU on the gate
         self.activation = act
         self.gate_act = ops.GateAct(act, float(spec.params.get("limit") or 0.0), float(spec.params.get("swish_alpha", 1.702)))
         if act == "clamped_swish" and not self.gate_act.limit > 0:

@@ -5,7 +5,12 @@ One part, every mechanism a parameter, so that a design picks the ones it has:
 ``qkv_bias``          biases on q, k and v, added in the projection
 ``qk_norm``           None; "projection": q as one vector of all its heads (and k alike) through an RMS norm
                       with weights before the rotation; "head_unit": every q and k head divided by its root
-                      mean square after the rotation
+                      mean square after the rotation; "head": every q and k head (with two maps every map's part)
+                      through an RMS norm before the rotation, a weight of head_dim numbers for q and one for k
+``differential``      {"diff": d}: two score maps a head over the same values.  q and k heads are [map 1 | map 2] of
+                      head_dim numbers each; with A_1 and A_2 the maps' softmax outputs and lambda = exp(lq1 . lk1) -
+                      exp(lq2 . lk2) + d (one number, tensors ``lq1`` ...), the head's output is z = A_1 - lambda A_2
+                      divided by its root mean square and times 1 - d (before a gate)
 ``value_norm``        every value head divided by its root mean square; the cache holds it so
 ``position``          a ``rope_computed`` part (partial rotation, interleaved or half-split pairs, scaled
                       frequencies with an amplitude on cos and sin)
@@ -42,6 +47,10 @@ kinds of memory, the pages (``kv``) and a record with the projections of the las
 else is done to q, k and v (no bias, norm, rotation or mixing) the convolution's kernel stores k and v itself.  Scores, softmax weights,
 norms and angles are float32 whatever the engine's dtype is.  q | k | v (| gate) are one product.
 
+Two maps run as twice as many query heads over the same keys and values: a cached key is its two parts side by side, and a
+query stands beside zeros in the place of the other map's part.  The attention kernels combine neighbouring heads before
+anything is rounded.
+
 Kernels: in bfloat16 with head sizes 64 and 128, tensor cores (``attn_shaped``: prompt portions 128 rows a CTA,
 single tokens with their keys split over CTAs; mixed heads as one wider query a head, made where q is
 normalised; prompt portions of a design without mixed heads and sink: the plain attention's tcgen05 kernel, the
@@ -63,7 +72,7 @@ from .short_conv import ConvMemory, PagedMemory, filters
 
 _NAMES = {"q": "q", "k": "k", "v": "v", "o": "o", "q_bias": "q.b", "k_bias": "k.b", "v_bias": "v.b",
           "q_norm": "q.norm", "k_norm": "k.norm", "temperature": "temp", "mix": "talk", "gate": "g",
-          "sink": "sink", "distance_bias": "rel", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv"}
+          "lq1": "lq1", "lk1": "lk1", "lq2": "lq2", "lk2": "lk2", "sink": "sink", "distance_bias": "rel", "q_conv": "q.conv", "k_conv": "k.conv", "v_conv": "v.conv"}
 
 
 def distance_bucket(n: int, buckets: int, farthest: float) -> int:
@@ -108,13 +117,16 @@ class ModulatedAttention(Mixer):
         slopes = p.get("distance_slopes")
         self.distance_slopes = None if slopes is None else tuple(float(s) for s in slopes)
         self.conv = int(p.get("conv") or 0)
+        self.differential = None if not p.get("differential") else float(p["differential"]["diff"])
+        self.maps = 1 if self.differential is None else 2
+        self.pairs = None                # (two maps: the weight of the second comes with the tensors)
         self.mask = str(p.get("mask", "causal"))
         size = p.get("mask_size")
         self.mask_size = None if size is None else int(size)
         if self.num_heads % self.num_kv_heads:
             raise ValueError("modulated_attention: num_heads must be a multiple of num_kv_heads")
         if self.qk_norm not in ops.QK_NORM:
-            raise ValueError(f"modulated_attention: qk_norm {self.qk_norm!r}; built: projection, head_unit, None")
+            raise ValueError(f"modulated_attention: qk_norm {self.qk_norm!r}; built: projection, head_unit, head, None")
         if self.mask not in ops.ATTN_MASK:
             raise ValueError(f"modulated_attention: mask {self.mask!r}; built: {', '.join(ops.ATTN_MASK)}")
         if self.mask != "causal" and (self.mask_size is None or self.mask_size <= 0):
@@ -133,6 +145,12 @@ class ModulatedAttention(Mixer):
                              "are not built")
         if self.distance_slopes is not None and len(self.distance_slopes) != self.num_heads:
             raise ValueError("modulated_attention: distance_slopes are a number a head")
+        if self.maps == 2 and (self.head_mix or self.conv or self.channel_gate or self.head_temperature or self.sink
+                               or self.distance_bias is not None or self.distance_slopes is not None):
+            raise ValueError("modulated_attention: two maps with mixed heads, a convolution, a channel gate, a head "
+                             "temperature, a sink or a distance bias are not built")
+        if self.maps == 2 and self.qk_norm not in (None, "head", "head_unit"):
+            raise ValueError("modulated_attention: two maps go with a norm a head (or none)")
         if self.conv and self.qkv_bias:
             raise ValueError("modulated_attention: a convolution of projections with biases is not built")
         if not (0 <= self.conv <= 64):
@@ -144,8 +162,11 @@ class ModulatedAttention(Mixer):
                              "(rope_computed)")
         self.names = dict(_NAMES)
         self.names.update(dict(p.get("tensor_names") or {}))
-        self.q_width = self.num_heads * self.head_dim
-        self.k_width = self.num_kv_heads * self.head_dim
+        # what the kernels see: query heads (a map of a head each) and the width of a cached key
+        self.map_heads = self.num_heads * self.maps
+        self.key_dim = self.head_dim * self.maps
+        self.q_width = self.num_heads * self.key_dim
+        self.k_width = self.num_kv_heads * self.key_dim
         self.v_width = self.num_kv_heads * self.vdim
         self.o_width = self.num_heads * self.vdim
         self.gate_offset = self.q_width + self.k_width + self.v_width
@@ -177,6 +198,12 @@ class ModulatedAttention(Mixer):
         if self.qk_norm == "projection":
             d[nm["q_norm"]] = TensorDecl((self.q_width,), "norm")
             d[nm["k_norm"]] = TensorDecl((self.k_width,), "norm")
+        if self.qk_norm == "head":
+            d[nm["q_norm"]] = TensorDecl((self.head_dim,), "norm")
+            d[nm["k_norm"]] = TensorDecl((self.head_dim,), "norm")
+        if self.differential is not None:
+            for name in ("lq1", "lk1", "lq2", "lk2"):
+                d[nm[name]] = TensorDecl((self.head_dim,), "bias", std=0.1)
         if self.head_temperature:
             d[nm["temperature"]] = TensorDecl((self.num_heads,), "norm")
         if self.head_mix:
@@ -213,7 +240,11 @@ class ModulatedAttention(Mixer):
         def f32(name):
             return fetch(nm[name]).to(torch.float32).to(device).contiguous()
 
-        if self.qk_norm == "projection":
+        if self.differential is not None:
+            dot = {i: (fetch(nm[f"lq{i}"]).to(torch.float64) * fetch(nm[f"lk{i}"]).to(torch.float64)).sum() for i in (1, 2)}
+            weight = float(torch.exp(dot[1]) - torch.exp(dot[2])) + self.differential
+            self.pairs = ops.MapPairs(weight, 1.0 - self.differential, self.eps)
+        if self.qk_norm in ("projection", "head"):
             self.q_norm_w, self.k_norm_w = f32("q_norm"), f32("k_norm")
         if self.head_temperature:
             self.temperature = f32("temperature")
@@ -243,9 +274,9 @@ class ModulatedAttention(Mixer):
         return None if self.conv else self._pages()
 
     def _pages(self) -> PagedKVNeed:
-        return PagedKVNeed(self.num_kv_heads, self.head_dim,
+        return PagedKVNeed(self.num_kv_heads, self.key_dim,
                            self.mask_size if self.mask == "window" else None,
-                           None if self.vdim == self.head_dim else self.vdim,
+                           None if self.vdim == self.key_dim else self.vdim,
                            self.mask_size if self.mask == "chunk" else None,
                            self.keep_first if self.mask == "window" else 0)
 
@@ -253,9 +284,9 @@ class ModulatedAttention(Mixer):
         libs = ["core", "attn_mod"] + (["short_conv"] if self.conv else [])
         if self.w_in is not None and self.w_in.dtype == torch.bfloat16:
             libs.extend(["gemm_smallm", "gemm_stream", "gemm_tc"])
-            if self.head_dim in (64, 128) and self.vdim in (64, 128):
+            if self.key_dim in (64, 128) and self.vdim in (64, 128):
                 libs.append("attn_shaped")
-                if not self.head_mix and not self.sink and not self.extended and self.vdim == self.head_dim and self.mask != "chunk":
+                if not self.head_mix and not self.sink and not self.extended and self.vdim == self.key_dim and self.mask != "chunk":
                     libs.append("attn_tc")
         return libs
 
@@ -288,7 +319,7 @@ class ModulatedAttention(Mixer):
             cache, record = cache["kv"], cache["conv"]
         # bfloat16 with head sizes the tensor-core kernel takes: mixed heads become one wider query a head
         shaped = ops.attn_shaped_supported(
-            proj.dtype, self.num_kv_heads, self.head_dim, self.vdim, cache.page_size, proj.stride(0), self.head_mix)
+            proj.dtype, self.num_kv_heads, self.key_dim, self.vdim, cache.page_size, proj.stride(0), self.head_mix)
         mixed_q = None
         if shaped and self.head_mix:
             mixed_q = torch.empty((n, self.num_heads * self.num_kv_heads * self.head_dim), dtype=proj.dtype,
@@ -308,14 +339,18 @@ class ModulatedAttention(Mixer):
             if direct:
                 self._attend_any(shaped, attn, proj, None, gate, step, cache, fold, out_scale)
                 return
+        paired_q = None
+        if self.maps == 2:
+            paired_q = torch.empty((n, self.map_heads * self.key_dim), dtype=proj.dtype, device=proj.device)
         ops.qkv_norm_rotate_store(
             proj, self.b_in, step.positions, None if pos is None else pos.freq,
-            1.0 if pos is None else pos.amplitude, bool(pos is None or pos.interleaved), self.num_heads,
-            self.num_kv_heads, self.head_dim, self.vdim, self.qk_norm, self.q_norm_w, self.k_norm_w, self.value_norm,
+            1.0 if pos is None else pos.amplitude, bool(pos is None or pos.interleaved), self.map_heads,
+            self.num_kv_heads * self.maps, self.head_dim, self.vdim, self.qk_norm, self.q_norm_w, self.k_norm_w, self.value_norm,
             self.eps, cache.slot_map if cache.writable else None, cache.k, cache.v, cache.page_size, step.status,
             head_mix=self.mix if mixed_q is not None else None,
-            mix_temperature=self.temperature if (mixed_q is not None or fold) else None, mixed_q=mixed_q)
-        self._attend_any(shaped, attn, proj, mixed_q, gate, step, cache, fold, out_scale)
+            mix_temperature=self.temperature if (mixed_q is not None or fold) else None, mixed_q=mixed_q,
+            paired_q=paired_q)
+        self._attend_any(shaped, attn, proj if paired_q is None else paired_q, mixed_q, gate, step, cache, fold, out_scale)
 
     def _attend_any(self, shaped, attn, proj, mixed_q, gate, step, cache, fold, out_scale) -> None:
         if shaped:
@@ -331,13 +366,13 @@ class ModulatedAttention(Mixer):
     def attend(self, out, proj, gate, step, cache, out_scale: float = 1.0) -> None:
         """Any sizes, both dtypes, float32 arithmetic: a block a token."""
         ops.attention_modulated(out, proj, proj.stride(0), gate, cache.k, cache.v, cache.block_table,
-                                step.token_req, step.req_slot, step.positions, proj.shape[0], self.num_heads,
-                                self.num_kv_heads, self.head_dim, self.vdim, cache.page_size, self.mask,
+                                step.token_req, step.req_slot, step.positions, proj.shape[0], self.map_heads,
+                                self.num_kv_heads, self.key_dim, self.vdim, cache.page_size, self.mask,
                                 self.mask_size, self.sink, self.scale, self.temperature, self.mix, step.status,
                                 sink_values=self.sink_w, distance_bias=self.bias_by_distance,
                                 keep_first=self.keep_first, softcap=self.softcap,
                                 query_temperature=self.query_temperature, gate_channels=self.channel_gate,
-                                out_scale=out_scale, distance_slope=self.slopes)
+                                out_scale=out_scale, distance_slope=self.slopes, pairs=self.pairs)
 
     def attend_shaped(self, out, proj, mixed_q, gate, step, cache, temperature, out_scale: float = 1.0) -> None:
         """Tensor cores.  Single-token entries come first in a step: their keys are cut into parts of one or more
@@ -347,16 +382,16 @@ class ModulatedAttention(Mixer):
         plain by now (no mixed heads, no sink, causal or a window, values as wide as keys; a temperature is on the
         queries already) go to the tcgen05 kernel of the plain attention, which takes the head gate."""
         q = proj if mixed_q is None else mixed_q
-        group = self.num_heads // self.num_kv_heads
+        group = self.map_heads // self.num_kv_heads
         n_single = step.num_single
         n_rest = step.num_entries - n_single
-        tail = (self.num_heads, self.num_kv_heads, self.head_dim, self.vdim, cache.page_size, self.mask,
+        tail = (self.map_heads, self.num_kv_heads, self.key_dim, self.vdim, cache.page_size, self.mask,
                 self.mask_size, self.sink, self.scale, step.status)
         head = (out, q, q.stride(0), mixed_q is not None, gate, temperature, cache.k, cache.v,
                 cache.block_table)
         more = dict(sink_values=self.sink_w, distance_bias=self.bias_by_distance, keep_first=self.keep_first,
                     softcap=self.softcap, query_temperature=self.query_temperature, gate_channels=self.channel_gate,
-                    out_scale=out_scale, distance_slope=self.slopes)
+                    out_scale=out_scale, distance_slope=self.slopes, pairs=self.pairs)
         if n_single > 0:
             if self.mask == "causal":
                 stages = (int(step.max_kv_len) + 63) // 64 + 1
@@ -372,10 +407,10 @@ class ModulatedAttention(Mixer):
             nsplit = (stages + span - 1) // span
             ops.attn_shaped(*head, step.cu_q, step.ctx_len, step.req_slot, n_single, n_single * ((group + 127) // 128),
                             *tail, nsplit=nsplit, span=span, **more)
-        if (n_rest > 0 and mixed_q is None and temperature is None and not self.sink and self.vdim == self.head_dim
+        if (n_rest > 0 and mixed_q is None and temperature is None and not self.sink and self.vdim == self.key_dim
                 and not self.extended and out_scale == 1.0
                 and self.mask in ("causal", "window") and ops.TC_ENABLED
-                and ops.attn_prefill_tc_supported(proj.dtype, self.head_dim, cache.page_size, proj.stride(0), group)):
+                and ops.attn_prefill_tc_supported(q.dtype, self.key_dim, cache.page_size, q.stride(0), group)):
             window = self.mask_size if self.mask == "window" else None
             key = ("attn_prefill_tc", group, window)
             plan = step.scratch.get(key)
@@ -391,9 +426,9 @@ class ModulatedAttention(Mixer):
                     plan = (blocks, ops.attn_prefill_tc_splits(blocks, self.num_kv_heads, proj.device), 8)
                 step.scratch[key] = plan
             ops.attn_prefill_tc(out, proj, proj.stride(0), cache.k, cache.v, cache.block_table, step.cu_q[n_single:],
-                                step.ctx_len[n_single:], step.req_slot[n_single:], n_rest, plan[0], self.num_heads,
-                                self.num_kv_heads, self.head_dim, cache.page_size, window, self.scale, step.status,
-                                nsplit=plan[1], split_len=plan[2], gate=gate)
+                                step.ctx_len[n_single:], step.req_slot[n_single:], n_rest, plan[0], self.map_heads,
+                                self.num_kv_heads, self.key_dim, cache.page_size, window, self.scale, step.status,
+                                nsplit=plan[1], split_len=plan[2], gate=gate, pairs=self.pairs)
         elif n_rest > 0:
             key = ("attn_shaped", group)
             blocks = step.scratch.get(key)

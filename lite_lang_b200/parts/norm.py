@@ -12,7 +12,7 @@ from typing import Dict, Optional
 import torch
 
 from .. import ops
-from .base import Norm, Pending, ResidualCopy, StreamWrite, TensorDecl, register_part, settled, whole_output
+from .base import Norm, NormedOutput, Pending, ResidualCopy, StreamWrite, TensorDecl, register_part, settled, whole_output
 
 
 class RMSNorm(Norm):
@@ -160,6 +160,66 @@ class RMSNormF32Residual(Norm):
         return new, out
 
 
+class SandwichRMSNorm(RMSNormF32Residual):
+    """The same norm between sublayers whose outputs have norms of their own: what is pending is a ``NormedOutput``, and one
+    pass takes the output's norm, adds it to the residual and takes this norm of the sum."""
+
+    def kernel_libraries(self):
+        return ("core", "sandwich")
+
+    def add_forward(self, residual, delta, rows=None):
+        if residual.dtype != torch.float32:
+            raise TypeError("rms_norm_f32_sandwich: the residual stream of this norm is float32")
+        if delta is None or isinstance(delta, ResidualCopy):
+            delta = NormedOutput(None)
+        if not isinstance(delta, NormedOutput):
+            raise TypeError(f"rms_norm_f32_sandwich: a pending {type(delta).__name__} is not built")
+        n = residual.shape[0] if rows is None else rows.numel()
+        out = torch.empty((n, self.hidden_size), dtype=self.out_dtype, device=residual.device)
+        ops.sandwich_norm(out, residual, delta.y, delta.weight, delta.eps, delta.row, self.weight, self.eps, rows)
+        return out
+
+
+class OutputRMSNorm(Norm):
+    """RMS norm with a weight on a sublayer's output, on its way into a float32 residual: y / sqrt(mean(y^2) + eps) * w,
+    with ``scale_tensor`` times a second weight (a layer scale), folded into the first in float32.  The norm after it in
+    the model takes it in its own pass (``pending``); ``apply`` is for a product that reads the residual itself: it adds
+    what is pending and returns the residual rounded to the engine's dtype.  ``tensor``, ``scale_tensor``: full names."""
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.hidden_size = int(spec.params["hidden_size"])
+        self.eps = float(spec.params["eps"])
+        self.tensor = str(spec.params["tensor"])
+        self.scale_tensor = spec.params.get("scale_tensor")
+        self.weight: Optional[torch.Tensor] = None
+
+    def tensors(self) -> Dict[str, TensorDecl]:
+        names = [self.tensor] + ([self.scale_tensor] if self.scale_tensor else [])
+        return {n: TensorDecl((self.hidden_size,), "norm") for n in names}
+
+    def load(self, fetch, dtype, device) -> None:
+        w = fetch(self.tensor).to(torch.float32)
+        if self.scale_tensor:
+            w = w * fetch(self.scale_tensor).to(torch.float32)
+        self.weight = w.to(device).contiguous()
+
+    def kernel_libraries(self):
+        return ("core", "sandwich")
+
+    def pending(self, y: torch.Tensor) -> NormedOutput:
+        return NormedOutput(y, self.weight, self.eps)
+
+    @staticmethod
+    def apply(residual: torch.Tensor, delta: NormedOutput, dtype: torch.dtype) -> torch.Tensor:
+        copy = None if dtype == torch.float32 else torch.empty(residual.shape, dtype=dtype, device=residual.device)
+        ops.sandwich_norm(copy, residual, delta.y, delta.weight, delta.eps, delta.row, None, 0.0)
+        return residual if copy is None else copy
+
+    def forward(self, x, out=None):
+        raise TypeError("rms_norm_out norms a sublayer's output into the residual stream: use pending")
+
+
 class DynamicTanh(Norm):
     """Dynamic tanh: y = tanh(alpha * u) * w + b with a scalar alpha; no mean, no variance.
 
@@ -266,3 +326,5 @@ register_part("norm", "layer_norm_out", OutputLayerNorm)
 register_part("norm", "dynamic_tanh", DynamicTanh)
 register_part("norm", "layer_norm_f32", LayerNormF32Residual)
 register_part("norm", "rms_norm_f32", RMSNormF32Residual)
+register_part("norm", "rms_norm_f32_sandwich", SandwichRMSNorm)
+register_part("norm", "rms_norm_out", OutputRMSNorm)

@@ -70,7 +70,11 @@ class RotaryComputed(PositionEncoding):
     d(t) = rotary_dim ln(original / (2 pi t)) / (2 ln theta), lo = max(floor d(fast), 0), hi = min(ceil d(slow),
     rotary_dim - 1) and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), pair i turns at
     f_i / factor * r_i + f_i (1 - r_i); cos and sin are both multiplied by ``amplitude`` = 0.1 ln(factor) + 1
-    (an attention that uses this part reads it and hands it to its kernel)."""
+    (an attention that uses this part reads it and hands it to its kernel).
+
+    ``scaling`` with (``factor``, ``low``, ``high``, ``original``) instead goes by the wavelength l = 2 pi / f_i: f_i stays
+    where l < original / high, becomes f_i / factor where l > original / low, and in between (1 - s) f_i / factor + s f_i
+    with s = (original / l - low) / (high - low); no amplitude."""
 
     computed = True
     fuses_with_store = False
@@ -90,7 +94,13 @@ class RotaryComputed(PositionEncoding):
         self.amplitude = 1.0
         sc = spec.params.get("scaling")
         self.scaling = None
-        if sc:
+        self.by_wavelength = bool(sc) and "low" in sc
+        if self.by_wavelength:
+            self.scaling = {k: float(sc[k]) for k in ("factor", "low", "high", "original")}
+            if self.scaling["factor"] <= 0 or self.scaling["original"] <= 0 or not self.scaling["high"] > self.scaling["low"] > 0:
+                raise ValueError("rope_computed: scaling by wavelength needs a positive factor and original length and "
+                                 "high > low > 0")
+        elif sc:
             self.scaling = {k: float(sc[k]) for k in ("factor", "original", "fast", "slow")}
             if self.scaling["factor"] <= 0 or self.scaling["original"] <= 0 or self.theta <= 1.0:
                 raise ValueError("rope_computed: scaling needs a positive factor and original length, theta above 1")
@@ -101,7 +111,12 @@ class RotaryComputed(PositionEncoding):
         i = torch.arange(0, self.rot_dim // 2, dtype=torch.float64)
         f = torch.pow(torch.tensor(self.theta, dtype=torch.float64), -2.0 * i / max(self.rot_dim, 1))
         f = f / self.position_scale
-        if self.scaling is not None:
+        if self.by_wavelength:
+            sc = self.scaling
+            turns = sc["original"] * f / (2.0 * math.pi)        # original / wavelength
+            s = torch.clamp((turns - sc["low"]) / (sc["high"] - sc["low"]), 0.0, 1.0)
+            f = (1.0 - s) * f / sc["factor"] + s * f
+        elif self.scaling is not None:
             sc = self.scaling
 
             def turns(t: float) -> float:
