@@ -457,7 +457,7 @@ def run_ours(args):
 
 
 # ---------------------------------------------------------------------------------------------------------
-# --compare nevurax / redirax / lenuzen / rufisun / tusipel: that design beside Qwen2 at equal layer sizes (random weights)
+# --compare nevurax / redirax / lenuzen / rufisun / tusipel / muduvik: that design beside Qwen2 at equal layer sizes (random weights)
 # ---------------------------------------------------------------------------------------------------------
 def _nevurax_shape(width, heads, kv_heads, head, inter, vocab, layers, window, experts, top):
     """A Nevurax model whose layers are as large as a Qwen2 layer of the given sizes: the mixers have as many
@@ -556,8 +556,28 @@ def _tusipel_shape(width, heads, kv_heads, head, inter, vocab, layers, window, e
                        for i in range(layers)]}
 
 
+def _muduvik_shape(width, heads, kv_heads, head, inter, vocab, layers, window, experts, top):
+    """A Muduvik model whose layers are as large as a Qwen2 layer of the given sizes.  The layers take turns: the windowed
+    attention of two score maps (as many heads, values of the head size, keys of half of it a map: as many scores' products
+    as one map of whole heads), the latent attention without positions (a latent of four key heads, queries through a latent
+    of 3/4 of the width) and retention (as many heads of the same size, no feed-forward behind it); the other layers have
+    the gated feed-forward.  A per-token table of 128 numbers a layer.  No layer runs twice."""
+    dense = {"kind": "dense", "ff": inter}
+    attention = {"heads": heads, "kv_heads": kv_heads, "dim": head // 2, "vdim": head, "scale": (head // 2) ** -0.5,
+                 "diff": 0.5, "mask": {"size": window},
+                 "rot": {"base": 1e6, "dims": head // 2,
+                         "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 4096}}}
+    latent = {"heads": heads, "dim": head, "vdim": head, "kv_rank": 4 * head, "q_rank": 3 * width // 4 // 64 * 64,
+              "scale": head ** -0.5}
+    retention = {"heads": heads, "dim": head, "vdim": head, "rot": {"base": 1e6, "dims": head},
+                 "decay": [1.0 - 2.0 ** (-2 - 6 * h / max(heads - 1, 1)) for h in range(heads)]}
+    kinds = [("attention", attention, dense), ("latent_attention", latent, dense), ("retention", retention, None)]
+    return {"architecture": "Muduvik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "token_side": {"dim": 128},
+            "layers": [dict(zip(("type", "mixer", "mlp"), kinds[i % 3])) for i in range(layers)]}
+
+
 COMPARE_DESIGNS = {"nevurax": _nevurax_shape, "redirax": _redirax_shape, "lenuzen": _lenuzen_shape,
-                   "rufisun": _rufisun_shape, "tusipel": _tusipel_shape}
+                   "rufisun": _rufisun_shape, "tusipel": _tusipel_shape, "muduvik": _muduvik_shape}
 
 COMPARE_SIZES = {
     # name: (Qwen2 sizes, window of the latent attention, experts, top)
@@ -658,6 +678,8 @@ def run_compare(args):
         elif design_name == "tusipel":
             row["config"] = {design_name: {"window": window, "chunk": window, "experts": experts, "identity": 4, "top": top,
                                            "expert_ff": nev["layers"][-1]["mlp"]["expert"]["ff"] if layers > 1 else None}}
+        elif design_name == "muduvik":
+            row["config"] = {design_name: {"window": window, "side": 128, "ff": nev["layers"][0]["mlp"]["ff"]}}
         elif design_name == "lenuzen":
             row["config"] = {design_name: {"window": window, "chunk": window, "ff": nev["layers"][-1]["mlp"]["ff"]}}
         else:
@@ -772,9 +794,9 @@ def main():
                     help="with --only: the layer sizes of that workload's model instead of Qwen2-1.5B's")
     ap.add_argument("--design-only", action="store_true", dest="design_only",
                     help="with --compare: leave the Qwen2 arm out")
-    ap.add_argument("--against", default="", choices=["", "qwen2", "nevurax", "redirax", "lenuzen", "rufisun"],
+    ap.add_argument("--against", default="", choices=["", "qwen2", "nevurax", "redirax", "lenuzen", "rufisun", "tusipel"],
                     help="with --compare: the arm beside the design (default qwen2)")
-    ap.add_argument("--compare", default="", choices=["", "nevurax", "redirax", "lenuzen", "rufisun", "tusipel"],
+    ap.add_argument("--compare", default="", choices=["", "nevurax", "redirax", "lenuzen", "rufisun", "tusipel", "muduvik"],
                     help="instead of the headline measurement: prefill and decode of a few layers of that design beside "
                          "Qwen2 at equal layer sizes (random weights); --layers (default 4), --size, --kernels go with it")
     ap.add_argument("--size", default="", dest="shape_name", choices=[""] + sorted(COMPARE_SIZES),

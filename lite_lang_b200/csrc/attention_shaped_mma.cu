@@ -541,19 +541,29 @@ __global__ void __launch_bounds__(AS_THREADS) attn_shaped_kernel(const AttnShape
 // The parts of a single token's rows meet: out[h] = sum_z O_z 2^(m_z - M) / (sum_z l_z 2^(m_z - M) + sink 2^-M),
 // M the largest maximum (0 at least with a sink), times the head's gate.  How many parts a row has follows
 // from its position as in the first kernel.  One block a (entry, head), a thread a value channel.
+// One row's value of channel d: the lanes of a warp take a part's maximum and sum each (32 parts at a time), so a row costs
+// two trips to memory and not two for every part.
 template <int VD>
 __device__ __forceinline__ float as_join_row(const AttnShapedParams& p, int tok, int head, int parts, int d) {
   const float* src = p.part + ((size_t)tok * p.nh + head) * p.nsplit * (VD + 2);
+  const int lane = threadIdx.x & 31;
   const float sink_log2 = p.sink_val ? p.sink_val[head] * AS_LOG2E : 0.f;
   float M = p.sink ? sink_log2 : -INFINITY;
-  for (int zz = 0; zz < parts; ++zz) M = fmaxf(M, src[(size_t)zz * (VD + 2) + VD]);
+  for (int z0 = 0; z0 < parts; z0 += 32)
+    M = fmaxf(M, warp_max(z0 + lane < parts ? src[(size_t)(z0 + lane) * (VD + 2) + VD] : -INFINITY));
   float L = (p.sink && M > -INFINITY) ? as_exp2(sink_log2 - M) : 0.f, acc = 0.f;
-  for (int zz = 0; zz < parts; ++zz) {
-    const float* s = src + (size_t)zz * (VD + 2);
-    const float m = s[VD];
+  for (int z0 = 0; z0 < parts; z0 += 32) {
+    float m = -INFINITY, l = 0.f;
+    if (z0 + lane < parts) {
+      m = src[(size_t)(z0 + lane) * (VD + 2) + VD];
+      l = src[(size_t)(z0 + lane) * (VD + 2) + VD + 1];
+    }
     const float w = m > -INFINITY ? as_exp2(m - M) : 0.f;
-    L = fmaf(s[VD + 1], w, L);
-    acc = fmaf(s[d], w, acc);
+    L += warp_sum(l * w);
+    const int n = min(32, parts - z0);
+#pragma unroll 8
+    for (int z = 0; z < n; ++z)
+      acc = fmaf(src[(size_t)(z0 + z) * (VD + 2) + d], __shfl_sync(0xffffffffu, w, z), acc);
   }
   return (L > 0.f ? acc / L : 0.f) * p.out_scale;
 }

@@ -199,7 +199,9 @@ extern "C" int ll_sandwich_norm(int dtype, void* out, float* residual, const voi
 }
 
 // ---------------------------------------------------------------------------------------------------------
-template <typename T>
+// (VEC 4: rows of up to 4 x 256 x EN_PIECES numbers stay in registers)
+#define EN_PIECES 4
+template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 embed_norm_kernel(float* __restrict__ out, const T* __restrict__ table, const int* __restrict__ ids,
                   const float* __restrict__ w, float eps, int hidden, int vocab, int* status) {
@@ -212,6 +214,25 @@ embed_norm_kernel(float* __restrict__ out, const T* __restrict__ table, const in
   float* dst = out + (size_t)blockIdx.x * hidden;
   const T* src = table + (size_t)(ok ? id : 0) * hidden;
   float ss = 0.f;
+  if (VEC == 4) {
+    float4 v[EN_PIECES];
+#pragma unroll
+    for (int p = 0; p < EN_PIECES; ++p) {
+      const int i = 4 * (threadIdx.x + p * 256);
+      v[p] = (ok && i < hidden) ? sn_load4<T>(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += sn_sq(v[p]);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)hidden + eps);
+#pragma unroll
+    for (int p = 0; p < EN_PIECES; ++p) {
+      const int i = 4 * (threadIdx.x + p * 256);
+      if (i < hidden) {
+        const float4 g = sn_load4<float>(w + i);
+        sn_store4<float>(dst + i, make_float4(v[p].x * inv * g.x, v[p].y * inv * g.y, v[p].z * inv * g.z, v[p].w * inv * g.w));
+      }
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < hidden; i += blockDim.x) {
     const float v = ok ? to_f32<T>(src[i]) : 0.f;
     ss += v * v;
@@ -225,8 +246,16 @@ extern "C" int ll_embed_norm(int dtype, float* out, const void* table, const int
                              int num_tokens, int hidden, int vocab, int* status, cudaStream_t stream) {
   if (num_tokens <= 0) return 0;
   if (hidden <= 0 || vocab <= 0 || w == nullptr) return (int)cudaErrorInvalidValue;
-  LL_DISPATCH_DTYPE(dtype, ll_launch(embed_norm_kernel<T>, dim3(num_tokens), dim3(256), 0, stream, out, (const T*)table,
-                                     ids, w, eps, hidden, vocab, status));
+  const bool wide = hidden % 4 == 0 && hidden <= 4 * 256 * EN_PIECES &&
+                    ((uintptr_t)out | (uintptr_t)table | (uintptr_t)w) % 16 == 0;
+  LL_DISPATCH_DTYPE(dtype, {
+    if (wide)
+      ll_launch(embed_norm_kernel<T, 4>, dim3(num_tokens), dim3(256), 0, stream, out, (const T*)table, ids, w, eps, hidden,
+                vocab, status);
+    else
+      ll_launch(embed_norm_kernel<T, 1>, dim3(num_tokens), dim3(256), 0, stream, out, (const T*)table, ids, w, eps, hidden,
+                vocab, status);
+  });
   return LL_LAUNCH_RESULT();
 }
 
