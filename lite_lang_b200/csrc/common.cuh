@@ -198,6 +198,19 @@ static inline void ll_launch_cluster(void (*kernel)(KArgs...), dim3 grid, dim3 b
   cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(std::forward<Args>(args))...);
 }
 
+// Launch that starts when the kernel before has ended, whatever its size: for kernels of about one CTA an SM that run long.
+// Started early, such a grid's CTAs pile up on the SMs that the kernel before has left first.
+template <typename... KArgs, typename... Args>
+static inline void ll_launch_after(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
+                                   Args&&... args) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid;
+  cfg.blockDim = block;
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(std::forward<Args>(args))...);
+}
+
 template <typename... KArgs, typename... Args>
 static inline void ll_launch(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem, cudaStream_t stream,
                              Args&&... args) {

@@ -332,11 +332,12 @@ linear_attn_out_kernel(T* __restrict__ y, const float* __restrict__ o, const flo
   }
 }
 
+// long_walk: the step holds a portion of a prompt (the scan then starts after the kernel before, see ll_launch_after).
 extern "C" int ll_decay_scan(int dtype, const void* proj, long stride, int q_off, int k_off, int v_off,
                              const float* decay, float* state, long slot_stride, int num_slots, const int* cu_q,
                              const int* req_slot, float* o, int num_entries, int H, int dk, int dv, int write_state,
                              int* status, int hpg, const float* tok_decay, const float* tok_scale, const float* skip,
-                             cudaStream_t stream) {
+                             int long_walk, cudaStream_t stream) {
   if (num_entries <= 0) return 0;
   if (H <= 0 || dk <= 0 || dk > 256 || dv <= 0 || hpg <= 0 || H % hpg != 0 || (decay == nullptr && tok_decay == nullptr))
     return (int)cudaErrorInvalidValue;
@@ -346,10 +347,14 @@ extern "C" int ll_decay_scan(int dtype, const void* proj, long stride, int q_off
   const int esz = dtype == LL_DTYPE_F32 ? 4 : 2, ve = 16 / esz;
   const bool vec = ((uintptr_t)proj % 16) == 0 && (stride % ve) == 0 && (q_off % ve) == 0 && (k_off % ve) == 0 &&
                    (dk % ve) == 0;
-#define LA_LAUNCH(RR, VV)                                                                                          \
-  ll_launch(decay_scan_kernel<T, RR, VV>, grid, dim3(LA_THREADS), 0, stream, (const T*)proj, stride, q_off, k_off, \
-            v_off, decay, state, slot_stride, num_slots, cu_q, req_slot, o, H, dk, dv, write_state, status, hpg,   \
-            tok_decay, tok_scale, skip)
+#define LA_ARGS                                                                                                     \
+  grid, dim3(LA_THREADS), 0, stream, (const T*)proj, stride, q_off, k_off, v_off, decay, state, slot_stride, num_slots,  \
+      cu_q, req_slot, o, H, dk, dv, write_state, status, hpg, tok_decay, tok_scale, skip
+#define LA_LAUNCH(RR, VV)                                                  \
+  do {                                                                     \
+    if (long_walk) ll_launch_after(decay_scan_kernel<T, RR, VV>, LA_ARGS); \
+    else ll_launch(decay_scan_kernel<T, RR, VV>, LA_ARGS);                 \
+  } while (0)
   LL_DISPATCH_DTYPE(dtype, {
     if (vec) {
       if (R == 4) LA_LAUNCH(4, true);
@@ -362,6 +367,7 @@ extern "C" int ll_decay_scan(int dtype, const void* proj, long stride, int q_off
     }
   });
 #undef LA_LAUNCH
+#undef LA_ARGS
   return LL_LAUNCH_RESULT();
 }
 

@@ -1584,7 +1584,7 @@ def decay_scan(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, decay: Op
         c_int(v_off), _ptr(decay), _ptr(state), c_long(state.stride(0)), c_int(state.shape[0]), _ptr(step.cu_q),
         _ptr(step.req_slot), _ptr(o), c_int(step.num_entries), c_int(H), c_int(dk), c_int(dv),
         c_int(1 if write_state else 0), _ptr(step.status), c_int(heads_per_group), _ptr(token_decay),
-        _ptr(token_scale), _ptr(skip), _stream())
+        _ptr(token_scale), _ptr(skip), c_int(1 if o.shape[0] >= 4 * step.num_entries + 128 else 0), _stream())
 
 
 def ssd_prepare(proj: torch.Tensor, x_off: int, dt_off: int, conv_w: torch.Tensor, conv_b: Optional[torch.Tensor],
