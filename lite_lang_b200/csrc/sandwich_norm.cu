@@ -12,7 +12,9 @@
 // output norm (a layer scale) is part of wa.  Everything is float32; out is rounded once.
 //
 // One block a row.  The row stays in registers between the sums (four neighbouring values an access, P accesses a
-// thread, every load in flight before the first sum); sizes that do not fit that go through shared memory.
+// thread, every load in flight before the first sum); sizes that do not fit that go through shared memory.  With few rows
+// (EARLY) a row's latency counts: as many threads as give each one access, the weights asked for before the kernel before
+// has ended.  With many rows the weights are read where they are used, which leaves registers for more rows an SM.
 //
 // `embed_norm`: the start of such a stream, out[t] = table[ids[t]] / sqrt(mean^2 + eps) * w in float32.
 // `token_side_act`: g[t, j] <- gelu_tanh(g[t, j]) * table[ids[t], first + j] in place: a per-token table's part for one
@@ -38,7 +40,7 @@ template <> __device__ __forceinline__ void sn_store4<bf16>(bf16* p, float4 v) {
 }
 __device__ __forceinline__ float sn_sq(float4 v) { return (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w); }
 
-template <typename T, int P>
+template <typename T, int P, bool EARLY>
 __global__ void __launch_bounds__(512)
 sandwich_norm_kernel(T* __restrict__ out, float* __restrict__ residual, const T* __restrict__ y,
                      const float* __restrict__ partial, int parts, long part_stride, const float* __restrict__ wa,
@@ -46,15 +48,16 @@ sandwich_norm_kernel(T* __restrict__ out, float* __restrict__ residual, const T*
                      const int* __restrict__ rows, int write_residual) {
   __shared__ float scratch[32];
   const int tid = threadIdx.x, step = 4 * blockDim.x;
-  float4 a4[P], b4[P], c4[P];      // the weights do not depend on the kernel before
+  const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+  auto weight = [&](const float* w, int i) { return w != nullptr && i < hidden ? sn_load4<float>(w + i) : zero; };
+  float4 a4[EARLY ? P : 1], b4[EARLY ? P : 1], c4[EARLY ? P : 1];
+  if (EARLY) {                     // (the weights do not depend on the kernel before)
 #pragma unroll
-  for (int p = 0; p < P; ++p) {
-    const int i = 4 * tid + p * step;
-    a4[p] = b4[p] = c4[p] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (i < hidden) {
-      if (wa) a4[p] = sn_load4<float>(wa + i);
-      if (wb) b4[p] = sn_load4<float>(wb + i);
-      if (add) c4[p] = sn_load4<float>(add + i);
+    for (int p = 0; p < P; ++p) {
+      const int i = 4 * tid + p * step;
+      a4[p] = weight(wa, i);
+      b4[p] = weight(wb, i);
+      c4[p] = weight(add, i);
     }
   }
   LL_PDL_TRIGGER();
@@ -67,7 +70,7 @@ sandwich_norm_kernel(T* __restrict__ out, float* __restrict__ residual, const T*
 #pragma unroll
   for (int p = 0; p < P; ++p) {
     const int i = 4 * tid + p * step;
-    v[p] = x[p] = make_float4(0.f, 0.f, 0.f, 0.f);
+    v[p] = x[p] = zero;
     if (i < hidden) {
       x[p] = sn_load4<float>(res + i);
       if (y) v[p] = sn_load4<T>(y + (size_t)r * hidden + i);
@@ -93,12 +96,13 @@ sandwich_norm_kernel(T* __restrict__ out, float* __restrict__ residual, const T*
   ss = 0.f;
 #pragma unroll
   for (int p = 0; p < P; ++p) {
-    x[p].x += v[p].x * inv * a4[p].x + c4[p].x;
-    x[p].y += v[p].y * inv * a4[p].y + c4[p].y;
-    x[p].z += v[p].z * inv * a4[p].z + c4[p].z;
-    x[p].w += v[p].w * inv * a4[p].w + c4[p].w;
-    ss += sn_sq(x[p]);
     const int i = 4 * tid + p * step;
+    const float4 a = EARLY ? a4[EARLY ? p : 0] : weight(wa, i), c = EARLY ? c4[EARLY ? p : 0] : weight(add, i);
+    x[p].x += v[p].x * inv * a.x + c.x;
+    x[p].y += v[p].y * inv * a.y + c.y;
+    x[p].z += v[p].z * inv * a.z + c.z;
+    x[p].w += v[p].w * inv * a.w + c.w;
+    ss += sn_sq(x[p]);
     if (write_residual && i < hidden) sn_store4<float>(res + i, x[p]);
   }
   if (out == nullptr) return;
@@ -110,7 +114,10 @@ sandwich_norm_kernel(T* __restrict__ out, float* __restrict__ residual, const T*
     const int i = 4 * tid + p * step;
     if (i < hidden) {
       float4 u = x[p];
-      if (wb) u = make_float4(u.x * io * b4[p].x, u.y * io * b4[p].y, u.z * io * b4[p].z, u.w * io * b4[p].w);
+      if (wb) {
+        const float4 b = EARLY ? b4[EARLY ? p : 0] : weight(wb, i);
+        u = make_float4(u.x * io * b.x, u.y * io * b.y, u.z * io * b.z, u.w * io * b.w);
+      }
       sn_store4<T>(o + i, u);
     }
   }
@@ -168,20 +175,23 @@ extern "C" int ll_sandwich_norm(int dtype, void* out, float* residual, const voi
   const uintptr_t ptrs = (uintptr_t)out | (uintptr_t)residual | (uintptr_t)y | (uintptr_t)partial | (uintptr_t)wa |
                          (uintptr_t)add | (uintptr_t)wb;
   if (hidden % 4 == 0 && ptrs % 16 == 0 && part_stride % 4 == 0 && hidden <= 512 * 4 * 4) {
-    // few rows: a row's latency counts, so as many threads as give each one access; many rows: fewer, so that more
-    // blocks fit an SM side by side
     const int quads = hidden / 4;
-    int threads = n_out <= 296 ? 512 : 256;
-    while (threads > 64 && threads / 2 >= quads) threads >>= 1;
-    while (quads > 4 * threads) threads <<= 1;
-    const int pieces = (quads + threads - 1) / threads;
-#define SN_LAUNCH(P)                                                                                              \
-  ll_launch(sandwich_norm_kernel<T, P>, dim3(n_out), dim3(threads), 0, stream, (T*)out, residual, (const T*)y,     \
+    const bool early = n_out <= 296;
+    const int most = early ? 512 : 256;
+    int pieces = (quads + most - 1) / most;
+    pieces = pieces <= 2 ? pieces : pieces <= 4 ? 4 : 8;
+    const int threads = ((quads + pieces - 1) / pieces + 31) / 32 * 32;
+#define SN_LAUNCH(P, E)                                                                                           \
+  ll_launch(sandwich_norm_kernel<T, P, E>, dim3(n_out), dim3(threads), 0, stream, (T*)out, residual, (const T*)y,  \
             partial, parts, part_stride, wa, eps_a, add, wb, eps_b, hidden, rows, write_residual)
     LL_DISPATCH_DTYPE(dtype, {
-      if (pieces == 1) SN_LAUNCH(1);
-      else if (pieces == 2) SN_LAUNCH(2);
-      else SN_LAUNCH(4);
+      if (early && pieces == 1) SN_LAUNCH(1, true);
+      else if (early && pieces == 2) SN_LAUNCH(2, true);
+      else if (early) SN_LAUNCH(4, true);
+      else if (pieces == 1) SN_LAUNCH(1, false);
+      else if (pieces == 2) SN_LAUNCH(2, false);
+      else if (pieces == 4) SN_LAUNCH(4, false);
+      else SN_LAUNCH(8, false);
     });
 #undef SN_LAUNCH
     return LL_LAUNCH_RESULT();
